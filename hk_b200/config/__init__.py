@@ -1,5 +1,6 @@
 from .base import (ConfigError, ModelConfig, architecture_name, config_from_dict, load_config,
                    register_architecture, resolve_architecture, supported_architectures)
+from .gezavik import GezavikConfig
 from .kedanex import KedanexConfig
 from .mifolorn import MifolornConfig
 from .padodra import PadodraConfig
@@ -7,6 +8,6 @@ from .qwen3 import Qwen3Config
 from .zazulix import ZazulixConfig
 
 __all__ = [
-    "ConfigError", "KedanexConfig", "MifolornConfig", "ModelConfig", "PadodraConfig", "Qwen3Config", "ZazulixConfig", "architecture_name", "config_from_dict", "load_config",
+    "ConfigError", "GezavikConfig", "KedanexConfig", "MifolornConfig", "ModelConfig", "PadodraConfig", "Qwen3Config", "ZazulixConfig", "architecture_name", "config_from_dict", "load_config",
     "register_architecture", "resolve_architecture", "supported_architectures",
 ]

@@ -44,6 +44,8 @@ LIBRARIES: Dict[str, str] = {
     "attention_latent": "attention_latent.cu",   # attention over a compressed cache whose rows are wider than a flash head
     "gemm_heads": "gemm_heads.cu",     # one small tensor-core product per head (a latent attention's up-projections)
     "recurrent": "recurrent.cu",       # scans of the recurrent mixers (delta rules, minGRU, matrix memory, retention)
+    "short_conv": "short_conv.cu",     # the causal convolution over a request's last rows that some mixers put behind their projections
+    "state_space": "state_space.cu",   # the state-space recurrence (Mamba-2) and the gated norm behind it
     "routed": "routed.cu",             # a feed-forward of experts: route, sort, grouped products, combine
     "runtime": "runtime.cpp",          # host only: the cache's books (no GPU code, no CUDA headers)
 }

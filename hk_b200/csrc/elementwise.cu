@@ -93,16 +93,17 @@ HK_API int hk_embedding(const void* table, int table_dtype, const int* ids, floa
 }
 
 // ----------------------------------------------------------------------------- rms norm
-// out[r, :] = x[row(r), :] * rsqrt(mean(x^2) + eps) * w, with row(r) = rows ? rows[r] : r.
+// out[r, :] = x[row(r), :] * rsqrt(mean(x^2) + eps) * w, with row(r) = rows ? rows[r] : r; rows of x lie ldx floats apart
+// (x may be a column slice of a wider matrix).
 // The sum of squares runs in a fixed order (thread-strided partials, warp tree, then
 // warps in order), so a row's result does not depend on what else is in the batch.
 template <typename TO>
 __global__ void rms_norm_kernel(const float* __restrict__ x, const float* __restrict__ w,
-                                const int* __restrict__ rows, TO* __restrict__ out, int d, float eps) {
+                                const int* __restrict__ rows, TO* __restrict__ out, int d, long long ldx, float eps) {
   __shared__ float warp_part[32];
   __shared__ float inv_s;
   int r = blockIdx.x;
-  const float* src = x + (size_t)(rows ? rows[r] : r) * d;
+  const float* src = x + (size_t)(rows ? rows[r] : r) * ldx;
   float ss = 0.f;
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float v = src[i];
@@ -129,7 +130,7 @@ __global__ void rms_norm_kernel(const float* __restrict__ x, const float* __rest
 template <typename TO, int PER>
 __global__ void __launch_bounds__(256)
 rms_norm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, const int* __restrict__ rows,
-                    TO* __restrict__ out, int d, float eps) {
+                    TO* __restrict__ out, int d, long long ldx, float eps) {
   __shared__ float warp_part[8];
   __shared__ float inv_s;
   const int r = blockIdx.x;
@@ -143,7 +144,7 @@ rms_norm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, co
     if (c < chunks) g[k] = wv[c];
   }
   pdl_wait();
-  const float4* src = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[r] : r) * d);
+  const float4* src = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[r] : r) * ldx);
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
     const int c = threadIdx.x + k * 256;
@@ -186,30 +187,30 @@ rms_norm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, co
 }
 
 template <int PER>
-static int rms_norm_vec(const float* x, const float* w, const int* rows, void* out, int out_dtype, int n_out, int d, float eps,
-                        cudaStream_t s) {
+static int rms_norm_vec(const float* x, const float* w, const int* rows, void* out, int out_dtype, int n_out, int d, long long ldx,
+                        float eps, cudaStream_t s) {
   if (out_dtype == HK_F32)
-    return hk_launch_pdl(rms_norm_vec_kernel<float, PER>, dim3(n_out), dim3(256), 0, s, x, w, rows, (float*)out, d, eps);
+    return hk_launch_pdl(rms_norm_vec_kernel<float, PER>, dim3(n_out), dim3(256), 0, s, x, w, rows, (float*)out, d, ldx, eps);
   if (out_dtype == HK_BF16)
-    return hk_launch_pdl(rms_norm_vec_kernel<bf16, PER>, dim3(n_out), dim3(256), 0, s, x, w, rows, (bf16*)out, d, eps);
+    return hk_launch_pdl(rms_norm_vec_kernel<bf16, PER>, dim3(n_out), dim3(256), 0, s, x, w, rows, (bf16*)out, d, ldx, eps);
   return HK_ERR_UNSUPPORTED;
 }
 
 HK_API int hk_rms_norm(const float* x, const float* w, const int* rows, void* out, int out_dtype,
-                       int n_out, int d, float eps, void* stream) {
+                       int n_out, int d, long long ldx, float eps, void* stream) {
   if (n_out <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
-  if ((d & 3) == 0 && d >= 1024 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0) {
+  if ((d & 3) == 0 && (ldx & 3) == 0 && d >= 1024 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0) {
     const int chunks = d >> 2;
-    if (chunks <= 2 * 256) return rms_norm_vec<2>(x, w, rows, out, out_dtype, n_out, d, eps, s);
-    if (chunks <= 4 * 256) return rms_norm_vec<4>(x, w, rows, out, out_dtype, n_out, d, eps, s);
-    if (chunks <= 8 * 256) return rms_norm_vec<8>(x, w, rows, out, out_dtype, n_out, d, eps, s);
+    if (chunks <= 2 * 256) return rms_norm_vec<2>(x, w, rows, out, out_dtype, n_out, d, ldx, eps, s);
+    if (chunks <= 4 * 256) return rms_norm_vec<4>(x, w, rows, out, out_dtype, n_out, d, ldx, eps, s);
+    if (chunks <= 8 * 256) return rms_norm_vec<8>(x, w, rows, out, out_dtype, n_out, d, ldx, eps, s);
   }
   int threads = d >= 2048 ? 256 : 128;
   if (out_dtype == HK_F32)
-    rms_norm_kernel<float><<<n_out, threads, 0, s>>>(x, w, rows, (float*)out, d, eps);
+    rms_norm_kernel<float><<<n_out, threads, 0, s>>>(x, w, rows, (float*)out, d, ldx, eps);
   else if (out_dtype == HK_BF16)
-    rms_norm_kernel<bf16><<<n_out, threads, 0, s>>>(x, w, rows, (bf16*)out, d, eps);
+    rms_norm_kernel<bf16><<<n_out, threads, 0, s>>>(x, w, rows, (bf16*)out, d, ldx, eps);
   else
     return HK_ERR_UNSUPPORTED;
   return hk_launch_status();
@@ -524,6 +525,27 @@ HK_API int hk_swiglu(const float* gu, void* out, int out_dtype, int n, int F, in
   return HK_ERR_UNSUPPORTED;
 }
 
+// ----------------------------------------------------------------------------- an activation without a gate
+// out = factor * max(z, 0)^2, element by element.
+template <typename TO>
+__global__ void squared_relu_kernel(const float* __restrict__ z, TO* __restrict__ out, long long total, float factor) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const float r = fmaxf(z[i], 0.f);
+  out[i] = from_f32<TO>(factor * (r * r));
+}
+
+HK_API int hk_squared_relu(const float* z, void* out, int out_dtype, long long total, float factor, void* stream) {
+  if (total <= 0) return 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const dim3 grid((unsigned)((total + 255) / 256));
+  if (out_dtype == HK_F32) return hk_launch_pdl(squared_relu_kernel<float>, grid, dim3(256), 0, s, z, (float*)out, total, factor);
+  if (out_dtype == HK_BF16) return hk_launch_pdl(squared_relu_kernel<bf16>, grid, dim3(256), 0, s, z, (bf16*)out, total, factor);
+  return HK_ERR_UNSUPPORTED;
+}
+
 // ----------------------------------------------------------------------------- norm of a sublayer's output, added
 // residual[r, :] += y[r, :] * rsqrt(mean(y^2) + eps) * w: the norm AFTER a mixer or feed-forward of a layer that
 // norms both sides of its sublayers, fused with the residual sum (which stays fp32).  Same summation order as
@@ -819,8 +841,9 @@ HK_API int hk_sigmoid_gate(const void* x, int x_dtype, const float* gate, long l
 }
 
 // ----------------------------------------------------------------------------- latent attention: what a token brings
-// A mixer that caches one compressed vector per token instead of keys and values.  One warp per (token, item) of the fused
-// projection's fp32 output row [H query heads of (dn + dr) | r + dr compressed | ...] (row stride ld):
+// A mixer that caches one compressed vector per token instead of keys and values.  One warp per (token, item) of two
+// fp32 projection outputs, the query heads q[n, H (dn + dr)] (row stride ldq) and the compressed row kv[n, r + dr] (row
+// stride ldkv; both may be slices of one matrix):
 //   query head h: its first dn dims go unchanged to q_plain[t, h, :dn] (they are multiplied with the keys' up-projection
 //                 afterwards); its last dr dims are rotated by the token's position into q_full[t, h, r : r + dr];
 //   the compressed row: its first r dims are RMS-normed with `c_w` (the latent), its last dr dims are rotated (the one
@@ -829,7 +852,7 @@ HK_API int hk_sigmoid_gate(const void* x, int x_dtype, const float* gate, long l
 // magnitude factor.  With write_kv == 0 only the queries are produced.
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(const float* __restrict__ proj, long long ld, T* __restrict__ q_plain, T* __restrict__ q_full,
+latent_prep_kernel(const float* __restrict__ q, long long ldq, const float* __restrict__ kv, long long ldkv, T* __restrict__ q_plain, T* __restrict__ q_full,
                    const float* __restrict__ c_w, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                    int rot, int pairing, const int* __restrict__ positions, const int* __restrict__ slot_of_token,
                    const int* __restrict__ block_table, int table_stride, T* __restrict__ pages, int n, int H, int dn, int dr,
@@ -842,14 +865,13 @@ latent_prep_kernel(const float* __restrict__ proj, long long ld, T* __restrict__
   if (item >= (long long)n * items) return;
   const int t = (int)(item / items), it = (int)(item % items);
   const int pos = positions[t];
-  const float* row = proj + (size_t)t * ld;
   const int half = rot >> 1;
   const float* c = cos_t + (size_t)pos * half;
   const float* s = sin_t + (size_t)pos * half;
   const float* src;   // the dr dims to rotate
   T* dst;             // where they go
   if (it < H) {
-    const float* qh = row + (size_t)it * (dn + dr);
+    const float* qh = q + (size_t)t * ldq + (size_t)it * (dn + dr);
     T* qp = q_plain + ((size_t)t * H + it) * dn;
     for (int i = lane; i < dn; i += 32) qp[i] = from_f32<T>(qh[i]);
     src = qh + dn;
@@ -857,7 +879,7 @@ latent_prep_kernel(const float* __restrict__ proj, long long ld, T* __restrict__
   } else {
     const int page = block_table[(size_t)slot_of_token[t] * table_stride + pos / page_tokens];
     if (page < 0) return;   // the host never schedules this; keeps a stale table from writing out of bounds
-    const float* cp = row + (size_t)H * (dn + dr);
+    const float* cp = kv + (size_t)t * ldkv;
     T* out = pages + ((size_t)page * page_tokens + (pos % page_tokens)) * (r + dr);
     float ss = 0.f;
     for (int i = lane; i < r; i += 32) ss = fmaf(cp[i], cp[i], ss);
@@ -876,7 +898,7 @@ latent_prep_kernel(const float* __restrict__ proj, long long ld, T* __restrict__
   for (int i = rot + lane; i < dr; i += 32) dst[i] = from_f32<T>(src[i]);
 }
 
-HK_API int hk_latent_prep(const float* proj, long long ld, void* q_plain, void* q_full, int dtype, const float* c_w, float eps,
+HK_API int hk_latent_prep(const float* q, long long ldq, const float* kv, long long ldkv, void* q_plain, void* q_full, int dtype, const float* c_w, float eps,
                           const float* cos_t, const float* sin_t, int rot, int pairing, const int* positions,
                           const int* slot_of_token, const int* block_table, int table_stride, void* pages, int n, int H, int dn,
                           int dr, int r, int page_tokens, int write_kv, void* stream) {
@@ -886,11 +908,11 @@ HK_API int hk_latent_prep(const float* proj, long long ld, void* q_plain, void* 
   const long long items = (long long)n * (H + (write_kv ? 1 : 0));
   const dim3 grid((unsigned)((items + 3) / 4)), block(128);
   if (dtype == HK_F32)
-    return hk_launch_pdl(latent_prep_kernel<float>, grid, block, 0, s, proj, ld, (float*)q_plain, (float*)q_full, c_w, eps, cos_t,
+    return hk_launch_pdl(latent_prep_kernel<float>, grid, block, 0, s, q, ldq, kv, ldkv, (float*)q_plain, (float*)q_full, c_w, eps, cos_t,
                          sin_t, rot, pairing, positions, slot_of_token, block_table, table_stride, (float*)pages, n, H, dn, dr, r,
                          page_tokens, write_kv);
   if (dtype == HK_BF16)
-    return hk_launch_pdl(latent_prep_kernel<bf16>, grid, block, 0, s, proj, ld, (bf16*)q_plain, (bf16*)q_full, c_w, eps, cos_t,
+    return hk_launch_pdl(latent_prep_kernel<bf16>, grid, block, 0, s, q, ldq, kv, ldkv, (bf16*)q_plain, (bf16*)q_full, c_w, eps, cos_t,
                          sin_t, rot, pairing, positions, slot_of_token, block_table, table_stride, (bf16*)pages, n, H, dn, dr, r,
                          page_tokens, write_kv);
   return HK_ERR_UNSUPPORTED;

@@ -161,7 +161,7 @@ def stream_wanted(M: int, N: int, K: int) -> bool:
 
 def run_stream(a, w, out, epilogue: int, ldo: int, limit: float = 0.0, slope: float = 1.0) -> bool:
     """The persistent streaming kernel; epilogue 0 store, 1 add, 2 silu(gate) * up (3: tanh gelu; 4: the clamped form with
-    its limit and slope) over w = [gate rows | up rows]."""
+    its limit and slope) over w = [gate rows | up rows], 5 slope * max(z, 0)^2 in bf16."""
     from . import ops
     M, K = a.shape
     N = w.shape[0]
@@ -176,6 +176,10 @@ def run_stream(a, w, out, epilogue: int, ldo: int, limit: float = 0.0, slope: fl
         code = lib.hk_gemm_stream_clamped(_ptr(a), _ptr(w), _ptr(out), M, N, K, ctypes.c_longlong(ldo),
                                           stream_row_warps(N, _sms(a.device)), _ptr(ws), _ptr(ct), _ptr(status_flag(a.device)),
                                           _stream_ctas, ctypes.c_float(limit), ctypes.c_float(slope), _stream())
+    elif epilogue == 5:
+        code = lib.hk_gemm_stream_sqrelu(_ptr(a), _ptr(w), _ptr(out), M, N, K, ctypes.c_longlong(ldo),
+                                         stream_row_warps(N, _sms(a.device)), _ptr(ws), _ptr(ct), _ptr(status_flag(a.device)),
+                                         _stream_ctas, ctypes.c_float(slope), _stream())
     else:
         code = lib.hk_gemm_stream(_ptr(a), _ptr(w), _ptr(out), M, N, K, ctypes.c_longlong(ldo), epilogue,
                                   stream_row_warps(N, _sms(a.device)),
@@ -262,11 +266,49 @@ def run_swiglu(a, w_gate_up, out, choice: Optional[str] = None, act: int = 0, li
     return True
 
 
+def run_squared_relu(a, w, out, factor: float, choice: Optional[str] = None) -> bool:
+    """out (bf16 [M, N]) = factor * max(a w^T, 0)^2 in the epilogue of the product that `run` would take for the shape.
+    False when no tensor-core kernel takes it."""
+    from . import ops
+    M, K = a.shape
+    N = w.shape[0]
+    if not _aligned(a, w):
+        return False
+    if choice == "stream" or (choice is None and stream_wanted(M, N, K)):
+        if run_stream(a, w, out, 5, N, slope=factor):
+            return True
+        if choice == "stream":
+            return False
+    if choice == "smallm" or (choice is None and M <= SMALL_M_AUTO):
+        if M > SMALL_M:
+            return False
+        lib = build.load("gemm_smallm")
+        code = lib.hk_gemm_smallm_sqrelu(_ptr(a), _ptr(w), _ptr(out), M, N, K, ctypes.c_longlong(N), row_tiles(M, N, a.device),
+                                         ctypes.c_float(factor), _stream())
+        if code == _UNSUPPORTED:
+            return False
+        ops._check(code, "gemm+squared relu (small-M)")
+        return True
+    lib = build.load("gemm_tc")
+    bn, splits = tc_config(M, N, K, _sms(a.device))
+    partial = _tc_partial(lib, M, N, splits, a.device)
+    code = lib.hk_gemm_tc_sqrelu(_ptr(a), _ptr(w), _ptr(out), M, N, K, ctypes.c_longlong(N), bn, splits,
+                                 _ptr(partial) if splits > 1 else ctypes.c_void_p(0), _ptr(status_flag(a.device)),
+                                 ctypes.c_float(factor), _stream())
+    if code == _UNSUPPORTED:
+        return False
+    ops._check(code, "gemm+squared relu (tcgen05)")
+    return True
+
+
 GROUPED_ROWS = 128      # rows of a tile of the grouped tcgen05 product: an expert's rows start on a multiple of it
 
 
-def run_grouped(a, w, out, groups, gated: bool) -> bool:
-    """out[tile rows] = a[tile rows] w[groups[tile]]^T over tiles of 128 rows (`hk_gemm_tc_grouped`)."""
+def run_grouped(a, w, out, groups, gated: bool, act: int = 0, limit: float = 0.0, slope: float = 1.0) -> bool:
+    """out[tile rows] = a[tile rows] w[groups[tile]]^T over tiles of 128 rows (`hk_gemm_tc_grouped`); gated: act 0 (silu) or
+    2 (the clamped form) of the two halves."""
+    if gated and act not in (0, 2):
+        return False
     from . import ops
     M, K = a.shape
     E, N = int(w.shape[0]), int(w.shape[1])
@@ -275,8 +317,8 @@ def run_grouped(a, w, out, groups, gated: bool) -> bool:
         return False
     bn = min(256, -(-N // 32) * 32)
     lib = build.load("gemm_tc")
-    code = lib.hk_gemm_tc_grouped(_ptr(a), _ptr(w), _ptr(out), M, N, K, ctypes.c_longlong(out.shape[1]), 2 if gated else 0, bn, E,
-                                  _ptr(groups), _ptr(status_flag(a.device)), _stream())
+    code = lib.hk_gemm_tc_grouped(_ptr(a), _ptr(w), _ptr(out), M, N, K, ctypes.c_longlong(out.shape[1]), 2 + act if gated else 0, bn, E,
+                                  _ptr(groups), _ptr(status_flag(a.device)), ctypes.c_float(limit), ctypes.c_float(slope), _stream())
     if code == _UNSUPPORTED:
         return False
     ops._check(code, "grouped gemm (tcgen05)")

@@ -9,7 +9,8 @@
 // a, of 2 for out), so either may be a column slice of wider rows; out is bf16 or fp32.  Each output element sums
 // k = 0..K-1 in one order whatever the batch, so a row's result does not depend on what else is in the step.
 // With `gate` (fp32 logits [M, >= heads * N], row stride gate_ld, head h at column h * N) the result is multiplied by
-// sigmoid(gate) in the epilogue: a mixer's output gate without a kernel of its own.
+// gate_scale * sigmoid(gate) in the epilogue: a mixer's output gate without a kernel of its own.  With gate_heads = 1 the
+// gate has one number per head (logits [M, >= heads], head h at column h).
 #include "common.cuh"
 
 namespace {
@@ -46,7 +47,7 @@ template <typename TO>
 __global__ void __launch_bounds__(128)
 gemm_heads_mma_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, TO* __restrict__ out, int M, int N, int K,
                       long long lda, long long a_head, long long ldo, long long o_head, const float* __restrict__ gate,
-                      long long gate_ld) {
+                      long long gate_ld, int gate_heads, float gate_scale) {
   __shared__ __align__(16) bf16 As[2][BM][LDS];
   __shared__ __align__(16) bf16 Ws[2][BN][LDS];
   pdl_launch_dependents();
@@ -103,11 +104,12 @@ gemm_heads_mma_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, TO
     const int gm = m0 + warp * 16 + qr + 8 * i;
     if (gm >= M) continue;
     TO* o = out + (size_t)gm * ldo;
-    const float* gr = gate ? gate + (size_t)gm * gate_ld + (size_t)h * N : nullptr;
+    const float* gr = gate && !gate_heads ? gate + (size_t)gm * gate_ld + (size_t)h * N : nullptr;
+    const float head_gate = gate ? (gate_heads ? gate_scale / (1.0f + expf(-gate[(size_t)gm * gate_ld + h])) : gate_scale) : 1.0f;
 #pragma unroll
     for (int n = 0; n < BN / 8; ++n) {
       const int gn = n0 + n * 8 + 2 * qt;
-      float x = acc[n][2 * i], y = acc[n][2 * i + 1];
+      float x = acc[n][2 * i] * head_gate, y = acc[n][2 * i + 1] * head_gate;
       if (gr) {
         if (gn < N) x /= 1.0f + expf(-gr[gn]);
         if (gn + 1 < N) y /= 1.0f + expf(-gr[gn + 1]);
@@ -123,7 +125,8 @@ gemm_heads_mma_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, TO
 // Refuses (HK_ERR_UNSUPPORTED) what the 16-byte copies and paired stores cannot take: K, lda or a_head no multiple of
 // 8, ldo or o_head odd, operands not 16-byte (out: 8-byte for fp32, 4-byte for bf16) aligned.
 HK_API int hk_gemm_heads_mma(const void* a, const void* w, void* out, int out_dtype, int M, int N, int K, int heads, long long lda,
-                             long long a_head, long long ldo, long long o_head, const float* gate, long long gate_ld, void* stream) {
+                             long long a_head, long long ldo, long long o_head, const float* gate, long long gate_ld, int gate_heads,
+                             float gate_scale, void* stream) {
   if (M <= 0 || N <= 0 || heads <= 0) return 0;
   if (K <= 0 || (K & 7) || (lda & 7) || (a_head & 7) || (ldo & 1) || (o_head & 1)) return HK_ERR_UNSUPPORTED;
   if (((uintptr_t)a & 15) || ((uintptr_t)w & 15) || ((uintptr_t)out & (out_dtype == HK_F32 ? 7 : 3))) return HK_ERR_UNSUPPORTED;
@@ -132,9 +135,9 @@ HK_API int hk_gemm_heads_mma(const void* a, const void* w, void* out, int out_dt
   cudaStream_t s = (cudaStream_t)stream;
   if (out_dtype == HK_F32)
     return hk_launch_pdl(gemm_heads_mma_kernel<float>, grid, dim3(128), 0, s, (const bf16*)a, (const bf16*)w, (float*)out, M, N, K, lda,
-                         a_head, ldo, o_head, gate, gate_ld);
+                         a_head, ldo, o_head, gate, gate_ld, gate_heads, gate_scale);
   if (out_dtype == HK_BF16)
     return hk_launch_pdl(gemm_heads_mma_kernel<bf16>, grid, dim3(128), 0, s, (const bf16*)a, (const bf16*)w, (bf16*)out, M, N, K, lda,
-                         a_head, ldo, o_head, gate, gate_ld);
+                         a_head, ldo, o_head, gate, gate_ld, gate_heads, gate_scale);
   return HK_ERR_UNSUPPORTED;
 }

@@ -7,7 +7,7 @@
 //     A lane loads 16 bytes (8 consecutive k) of w row g (and g + 8) and the same 8 k of token g; the two
 //     MMAs that consume them pair slot with slot, so any k order is fine as long as both sides agree;
 //   * the 8 partial sums meet in shared memory and are added in warp order (deterministic), then stored
-//     or added onto `out` (the residual sum).
+//     or added onto `out` (the residual sum), or narrowed behind a squared relu (factor * max(z, 0)^2 in bf16).
 // The activations are tiny and come from L2; tokens beyond M and rows beyond N are clamped on load and
 // skipped on store.  Needs K % 8 == 0 and 16-byte aligned a and w.
 //
@@ -33,10 +33,12 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 }
 
 // MT: token tiles of 8 (M <= 8*MT).  RT: row tiles of 16 per CTA.
-template <int MT, int RT, bool ADD>
+enum Mode { STORE = 0, ADD = 1, SQRELU = 2 };
+
+template <int MT, int RT, int MODE>
 __global__ void __launch_bounds__(SM_WARPS * 32)
-gemm_smallm_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, float* __restrict__ out, int M, int N, int K,
-                   long long ldo) {
+gemm_smallm_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, void* __restrict__ out, int M, int N, int K,
+                   long long ldo, float factor) {
   extern __shared__ float red[];   // [SM_WARPS][RT*16][MT*8]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
@@ -147,42 +149,61 @@ gemm_smallm_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, float
     float s = 0.f;
 #pragma unroll
     for (int wv = 0; wv < SM_WARPS; ++wv) s += red[(size_t)wv * ROWS * COLS + row * COLS + m];
-    float* o = out + (size_t)m * ldo + n0 + row;
-    *o = ADD ? *o + s : s;
+    if (MODE == SQRELU) {
+      const float r = fmaxf(s, 0.f);
+      reinterpret_cast<bf16*>(out)[(size_t)m * ldo + n0 + row] = __float2bfloat16_rn(factor * (r * r));
+      continue;
+    }
+    float* o = reinterpret_cast<float*>(out) + (size_t)m * ldo + n0 + row;
+    *o = MODE == ADD ? *o + s : s;
   }
 }
 
-template <int MT, int RT>
-int launch(const void* a, const void* w, float* out, int M, int N, int K, long long ldo, int add, cudaStream_t s) {
+template <int MT, int RT, int MODE>
+int launch_mode(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, float factor, cudaStream_t s) {
   const size_t smem = (size_t)SM_WARPS * RT * 16 * MT * 8 * sizeof(float);
-  static HkSmemCache allowed_store = {}, allowed_add = {};
-  if (int e = hk_allow_smem(gemm_smallm_kernel<MT, RT, false>, smem, allowed_store)) return e;
-  if (int e = hk_allow_smem(gemm_smallm_kernel<MT, RT, true>, smem, allowed_add)) return e;
+  static HkSmemCache allowed = {};
+  if (int e = hk_allow_smem(gemm_smallm_kernel<MT, RT, MODE>, smem, allowed)) return e;
   const unsigned grid = (unsigned)((N + RT * 16 - 1) / (RT * 16));
   // launched so that it may start while the kernel before it drains: its first weights are on their way before it
   // waits for that kernel's output (0.8 microseconds a launch, measured over a decode step)
-  if (add)
-    return hk_launch_pdl(gemm_smallm_kernel<MT, RT, true>, dim3(grid), dim3(SM_WARPS * 32), smem, s, (const bf16*)a, (const bf16*)w,
-                         out, M, N, K, ldo);
-  return hk_launch_pdl(gemm_smallm_kernel<MT, RT, false>, dim3(grid), dim3(SM_WARPS * 32), smem, s, (const bf16*)a, (const bf16*)w,
-                       out, M, N, K, ldo);
+  return hk_launch_pdl(gemm_smallm_kernel<MT, RT, MODE>, dim3(grid), dim3(SM_WARPS * 32), smem, s, (const bf16*)a, (const bf16*)w,
+                       out, M, N, K, ldo, factor);
+}
+
+template <int MT, int RT>
+int launch(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int mode, float factor, cudaStream_t s) {
+  if (mode == ADD) return launch_mode<MT, RT, ADD>(a, w, out, M, N, K, ldo, factor, s);
+  if (mode == SQRELU) return launch_mode<MT, RT, SQRELU>(a, w, out, M, N, K, ldo, factor, s);
+  return launch_mode<MT, RT, STORE>(a, w, out, M, N, K, ldo, factor, s);
 }
 
 }  // namespace
 
-// rt: row tiles of 16 per CTA (1, 2 or 4).  Refuses (HK_ERR_UNSUPPORTED) M > 64, K % 8 != 0, unaligned operands.
-HK_API int hk_gemm_smallm(const void* a, const void* w, float* out, int M, int N, int K, long long ldo, int add, int rt,
-                          void* stream) {
+static int gemm_smallm_run(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int mode, int rt, float factor,
+                           void* stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64 || K <= 0 || (K & 7) || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
   const int mt = M <= 8 ? 1 : M <= 16 ? 2 : M <= 32 ? 4 : 8;
 #define HK_CASE(MT, RT) \
-  if (mt == MT && rt == RT) return launch<MT, RT>(a, w, out, M, N, K, ldo, add, s);
+  if (mt == MT && rt == RT) return launch<MT, RT>(a, w, out, M, N, K, ldo, mode, factor, s);
   HK_CASE(1, 1) HK_CASE(1, 2) HK_CASE(1, 4)
   HK_CASE(2, 1) HK_CASE(2, 2) HK_CASE(2, 4)
   HK_CASE(4, 1) HK_CASE(4, 2)
   HK_CASE(8, 1) HK_CASE(8, 2)
 #undef HK_CASE
   return HK_ERR_UNSUPPORTED;
+}
+
+// rt: row tiles of 16 per CTA (1, 2 or 4).  Refuses (HK_ERR_UNSUPPORTED) M > 64, K % 8 != 0, unaligned operands.
+HK_API int hk_gemm_smallm(const void* a, const void* w, float* out, int M, int N, int K, long long ldo, int add, int rt,
+                          void* stream) {
+  return gemm_smallm_run(a, w, out, M, N, K, ldo, add ? ADD : STORE, rt, 1.0f, stream);
+}
+
+// out bf16 [M, N] = factor * max(a w^T, 0)^2; everything else as above.
+HK_API int hk_gemm_smallm_sqrelu(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int rt, float factor,
+                                 void* stream) {
+  return gemm_smallm_run(a, w, out, M, N, K, ldo, SQRELU, rt, factor, stream);
 }

@@ -48,14 +48,19 @@ constexpr uint32_t WAIT_LIMIT = 1u << 20;
 constexpr int SMEM_BUDGET = 152 * 1024;
 constexpr int SMEM_BUDGET_WIDE = 200 * 1024;     // 17 to 32 rows: a stage is 48 KB, and three must fit
 
-enum Epilogue { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_GEGLU = 3, EPI_CLAMPGLU = 4 };
+enum Epilogue { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_GEGLU = 3, EPI_CLAMPGLU = 4, EPI_SQRELU = 5 };
 // The first two gated epilogues differ in the gate's activation alone: silu, or the tanh form of gelu, which is
 // g * sigmoid(2 * sqrt(2 / pi) * (g + 0.044715 g^3)).  The third clamps both halves first: with g = min(gate, limit) and
 // u = clamp(up, -limit, limit) it gives g * sigmoid(slope * g) * (u + 1); limit and slope travel as kernel arguments.
+// EPI_SQRELU has no gate: slope * max(z, 0)^2 narrowed to bf16 (slope is a factor on the result).
 #define IS_GLU(e) ((e) == EPI_SWIGLU || (e) == EPI_GEGLU || (e) == EPI_CLAMPGLU)
 struct GluParams {
   float limit, slope;
 };
+__device__ __forceinline__ bf16 squared_relu(float z, GluParams gp) {
+  const float r = fmaxf(z, 0.f);
+  return __float2bfloat16_rn(gp.slope * (r * r));
+}
 template <int EPI>
 __device__ __forceinline__ float glu_pair(float g, float u, GluParams gp) {
   if (EPI == EPI_CLAMPGLU) {
@@ -275,8 +280,12 @@ __device__ __forceinline__ void consume_units(const Sched& sc, uint32_t i_base, 
           for (int e = tid; e < BN * COLS; e += CONSUMERS * 32) {
             const int m = e / BN, row = e % BN;
             if (m >= M || n0 + row >= N) continue;
-            float* o = reinterpret_cast<float*>(out) + (size_t)m * ldo + n0 + row;
             const float v = value(e);
+            if (EPI == EPI_SQRELU) {
+              reinterpret_cast<bf16*>(out)[(size_t)m * ldo + n0 + row] = squared_relu(v, gp);
+              continue;
+            }
+            float* o = reinterpret_cast<float*>(out) + (size_t)m * ldo + n0 + row;
             *o = EPI == EPI_ADD ? *o + v : v;
           }
         }
@@ -465,6 +474,7 @@ int launch_epi(int epilogue, const void* a, const void* w, void* out, int M, int
   if (epilogue == EPI_ADD) return launch<RW, MT, EPI_ADD>(a, w, out, M, N, K, ldo, workspace, counters, status, max_ctas, s);
   if (epilogue == EPI_GEGLU) return launch<RW, MT, EPI_GEGLU>(a, w, out, M, N, K, ldo, workspace, counters, status, max_ctas, s);
   if (epilogue == EPI_CLAMPGLU) return launch<RW, MT, EPI_CLAMPGLU>(a, w, out, M, N, K, ldo, workspace, counters, status, max_ctas, s, gp);
+  if (epilogue == EPI_SQRELU) return launch<RW, MT, EPI_SQRELU>(a, w, out, M, N, K, ldo, workspace, counters, status, max_ctas, s, gp);
   return launch<RW, MT, EPI_SWIGLU>(a, w, out, M, N, K, ldo, workspace, counters, status, max_ctas, s);
 }
 
@@ -482,7 +492,7 @@ static int gemm_stream_run(const void* a, const void* w, void* out, int M, int N
                            float* workspace, int* counters, int* status, int max_ctas, GluParams gp, void* stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 32 || K <= 0 || (K & 63) || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return HK_ERR_UNSUPPORTED;
-  if (epilogue < 0 || epilogue > 4 || (IS_GLU(epilogue) && (rw < 1 || N % (16 * rw)))) return HK_ERR_UNSUPPORTED;
+  if (epilogue < 0 || epilogue > EPI_SQRELU || (IS_GLU(epilogue) && (rw < 1 || N % (16 * rw)))) return HK_ERR_UNSUPPORTED;
   if (workspace == nullptr || counters == nullptr || status == nullptr) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
   const int mt = M <= 8 ? 1 : M <= 16 ? 2 : 4;
@@ -497,7 +507,7 @@ static int gemm_stream_run(const void* a, const void* w, void* out, int M, int N
 
 HK_API int hk_gemm_stream(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int epilogue, int rw,
                           float* workspace, int* counters, int* status, int max_ctas, void* stream) {
-  if (epilogue == EPI_CLAMPGLU) return HK_ERR_UNSUPPORTED;      // that one needs its two numbers: hk_gemm_stream_clamped
+  if (epilogue > EPI_GEGLU) return HK_ERR_UNSUPPORTED;      // those need their numbers: hk_gemm_stream_clamped, hk_gemm_stream_sqrelu
   return gemm_stream_run(a, w, out, M, N, K, ldo, epilogue, rw, workspace, counters, status, max_ctas, GluParams{0.f, 1.f}, stream);
 }
 
@@ -507,6 +517,13 @@ HK_API int hk_gemm_stream_clamped(const void* a, const void* w, void* out, int M
                                   float* workspace, int* counters, int* status, int max_ctas, float limit, float slope,
                                   void* stream) {
   return gemm_stream_run(a, w, out, M, N, K, ldo, EPI_CLAMPGLU, rw, workspace, counters, status, max_ctas, GluParams{limit, slope},
+                         stream);
+}
+
+// The product with a squared relu and no gate (epilogue 5): out bf16 [M, N] = factor * max(a w^T, 0)^2.
+HK_API int hk_gemm_stream_sqrelu(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int rw,
+                                 float* workspace, int* counters, int* status, int max_ctas, float factor, void* stream) {
+  return gemm_stream_run(a, w, out, M, N, K, ldo, EPI_SQRELU, rw, workspace, counters, status, max_ctas, GluParams{0.f, factor},
                          stream);
 }
 

@@ -40,14 +40,19 @@ constexpr int RING_BYTES = 227 * 1024 - 2 * 1024;   // what is left of an SM's s
 constexpr uint32_t TMEM_COLS = 2 * MAX_BN;
 constexpr uint32_t WAIT_LIMIT = 1u << 24;
 
-enum Epilogue { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_GEGLU = 3, EPI_CLAMPGLU = 4 };
+enum Epilogue { EPI_STORE = 0, EPI_ADD = 1, EPI_SWIGLU = 2, EPI_GEGLU = 3, EPI_CLAMPGLU = 4, EPI_SQRELU = 5 };
 // The first two gated epilogues differ in the gate's activation alone: silu, or the tanh form of gelu, which is
 // g * sigmoid(2 * sqrt(2 / pi) * (g + 0.044715 g^3)).  The third clamps both halves first: with g = min(gate, limit) and
 // u = clamp(up, -limit, limit) it gives g * sigmoid(slope * g) * (u + 1); limit and slope travel as kernel arguments.
+// EPI_SQRELU has no gate: slope * max(z, 0)^2 narrowed to bf16 (slope is a factor on the result).
 #define IS_GLU(e) ((e) == EPI_SWIGLU || (e) == EPI_GEGLU || (e) == EPI_CLAMPGLU)
 struct GluParams {
   float limit, slope;
 };
+__device__ __forceinline__ bf16 squared_relu(float z, GluParams gp) {
+  const float r = fmaxf(z, 0.f);
+  return __float2bfloat16_rn(gp.slope * (r * r));
+}
 template <int EPI>
 __device__ __forceinline__ float glu_pair(float g, float u, GluParams gp) {
   if (EPI == EPI_CLAMPGLU) {
@@ -207,6 +212,32 @@ __device__ __forceinline__ void add_chunk_prefetched(uint32_t taddr, float* o, i
 __device__ __forceinline__ void load_chunk(const float* o, int c0, float4* y) {
 #pragma unroll
   for (int j = 0; j < 8; ++j) y[j] = *reinterpret_cast<const float4*>(o + c0 + 4 * j);
+}
+
+// W columns as W bf16 outputs slope * max(z, 0)^2.
+template <int W>
+__device__ __forceinline__ void sqrelu_chunk(uint32_t taddr, bf16* o, int c0, int n_out, bool row_ok, bool vec_ok, GluParams gp) {
+  uint32_t v[W];
+  tmem_ld<W>(taddr + (uint32_t)c0, v);
+  tmem_ld_wait();
+  if (!row_ok) return;
+  if (c0 + W <= n_out && vec_ok) {
+#pragma unroll
+    for (int j = 0; j < W; j += 8) {
+      uint32_t packed[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        __nv_bfloat162 p;
+        p.x = squared_relu(__uint_as_float(v[j + 2 * e]), gp);
+        p.y = squared_relu(__uint_as_float(v[j + 2 * e + 1]), gp);
+        packed[e] = *reinterpret_cast<uint32_t*>(&p);
+      }
+      *reinterpret_cast<uint4*>(o + c0 + j) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+    }
+  } else {
+    for (int j = 0; j < W; ++j)
+      if (c0 + j < n_out) o[c0 + j] = squared_relu(__uint_as_float(v[j]), gp);
+  }
 }
 
 // W gate columns at c0 and their up columns `h` further on -> W bf16 outputs silu(gate) * up.
@@ -403,6 +434,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll 1
         for (; c0 + 32 <= h; c0 += 32) swiglu_chunk<32, EPI>(taddr, o, c0, h, n_out, row_ok, vec_ok, gp);
         if (c0 < h) swiglu_chunk<16, EPI>(taddr, o, c0, h, n_out, row_ok, vec_ok, gp);
+      } else if (EPI == EPI_SQRELU) {
+        bf16* o = reinterpret_cast<bf16*>(out) + (size_t)row * ldo + nt * bn;
+        const int n_out = N - nt * bn;
+        const bool vec_ok = (ldo & 7) == 0 && ((nt * bn) & 7) == 0;
+        int c0 = 0;
+#pragma unroll 1
+        for (; c0 + 32 <= bn; c0 += 32) sqrelu_chunk<32>(taddr, o, c0, n_out, row_ok, vec_ok, gp);
+        if (c0 < bn) sqrelu_chunk<16>(taddr, o, c0, n_out, row_ok, vec_ok, gp);
       } else {
         const int n0 = nt * bn;
         float* o = reinterpret_cast<float*>(out) + (size_t)row * ldo + n0;
@@ -483,17 +522,18 @@ int sm_count() {
 }
 
 // Adds the K slices of a split product in slice order.  mode 0: out fp32 = sum; 1: out fp32 += sum;
-// 2 (silu), 3 (tanh gelu) and 4 (clamped): out bf16 [M, N/2] = act(gate) * up, the partial sums' columns in tiles of [bn / 2 gates | their bn / 2 ups].
+// 2 (silu), 3 (tanh gelu) and 4 (clamped): out bf16 [M, N/2] = act(gate) * up, the partial sums' columns in tiles of [bn / 2 gates | their bn / 2 ups];
+// 5: out bf16 [M, N] = slope * max(sum, 0)^2.
 template <int MODE>
 __global__ void splitk_reduce_kernel(const float* __restrict__ partial, void* __restrict__ out, int M, int N, long long ldo,
                                      int splits, int bn, GluParams gp) {
-  const long long total = MODE >= 2 ? (long long)M * (N / 2) : (long long)M * N;
+  const long long total = IS_GLU(MODE) ? (long long)M * (N / 2) : (long long)M * N;
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   pdl_launch_dependents();
   pdl_wait();          // the partial sums come from the kernel before
   if (i >= total) return;
   const size_t slice = slice_floats(M, N);
-  if (MODE >= 2) {
+  if (IS_GLU(MODE)) {
     const int F = N / 2;
     const int m = (int)(i / F), j = (int)(i % F);
     const int h = bn >> 1;
@@ -508,6 +548,10 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ partial, void* __
     const int m = (int)(i / N), n = (int)(i % N);
     float sum = 0.f;
     for (int s = 0; s < splits; ++s) sum += partial[s * slice + i];
+    if (MODE == EPI_SQRELU) {
+      reinterpret_cast<bf16*>(out)[(size_t)m * ldo + n] = squared_relu(sum, gp);
+      return;
+    }
     float* o = reinterpret_cast<float*>(out) + (size_t)m * ldo + n;
     *o = MODE == 1 ? *o + sum : sum;
   }
@@ -554,7 +598,7 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mw, void* out, int M, int N
   // dependent launches (measured over decode steps of 24 and 64 rows: 1 % faster; the kernels after this one set up while it drains)
   int code = hk_launch_pdl(gemm_tc_kernel<EPI>, dim3(grid), dim3(NUM_THREADS), smem, s, ma, mw, out, M, N, K, ldo, bn, stages, splits, partial, status, groups, gp);
   if (code != 0 || splits <= 1) return code;
-  if (!IS_GLU(EPI) && (N & 3) == 0 && (ldo & 3) == 0 && ((uintptr_t)out & 15) == 0) {
+  if (EPI <= EPI_ADD && (N & 3) == 0 && (ldo & 3) == 0 && ((uintptr_t)out & 15) == 0) {
     const long long quads = (long long)M * (N / 4);
     return hk_launch_pdl(splitk_reduce_vec_kernel<EPI == EPI_ADD ? 1 : 0>, dim3((unsigned)((quads + 127) / 128)), dim3(128), 0, s,
                          (const float*)partial, reinterpret_cast<float*>(out), M, N, ldo, splits);
@@ -578,7 +622,7 @@ static int gemm_tc_run(const void* a, const void* w, void* out, int M, int N, in
                        int splits, float* partial, int* status, GluParams gp, void* stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K & 7) || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return HK_ERR_UNSUPPORTED;
-  if (epilogue < EPI_STORE || epilogue > EPI_CLAMPGLU) return HK_ERR_UNSUPPORTED;
+  if (epilogue < EPI_STORE || epilogue > EPI_SQRELU) return HK_ERR_UNSUPPORTED;
   if (bn < 16 || bn > MAX_BN || (bn & 15)) return HK_ERR_UNSUPPORTED;
   if (IS_GLU(epilogue) && ((N & 1) || (bn & 31))) return HK_ERR_UNSUPPORTED;
   if (splits < 1 || splits > (K + BK - 1) / BK || (splits > 1 && partial == nullptr)) return HK_ERR_UNSUPPORTED;
@@ -590,12 +634,13 @@ static int gemm_tc_run(const void* a, const void* w, void* out, int M, int N, in
   if (epilogue == EPI_ADD) return launch<EPI_ADD>(ma, mw, out, M, N, K, ldo, bn, splits, partial, status, s);
   if (epilogue == EPI_GEGLU) return launch<EPI_GEGLU>(ma, mw, out, M, N, K, ldo, bn, splits, partial, status, s);
   if (epilogue == EPI_CLAMPGLU) return launch<EPI_CLAMPGLU>(ma, mw, out, M, N, K, ldo, bn, splits, partial, status, s, nullptr, gp);
+  if (epilogue == EPI_SQRELU) return launch<EPI_SQRELU>(ma, mw, out, M, N, K, ldo, bn, splits, partial, status, s, nullptr, gp);
   return launch<EPI_SWIGLU>(ma, mw, out, M, N, K, ldo, bn, splits, partial, status, s);
 }
 
 HK_API int hk_gemm_tc(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int epilogue, int bn,
                       int splits, float* partial, int* status, void* stream) {
-  if (epilogue == EPI_CLAMPGLU) return HK_ERR_UNSUPPORTED;      // that one needs its two numbers: hk_gemm_tc_clamped
+  if (epilogue > EPI_GEGLU) return HK_ERR_UNSUPPORTED;      // those need their numbers: hk_gemm_tc_clamped, hk_gemm_tc_sqrelu
   return gemm_tc_run(a, w, out, M, N, K, ldo, epilogue, bn, splits, partial, status, GluParams{0.f, 1.f}, stream);
 }
 
@@ -606,17 +651,24 @@ HK_API int hk_gemm_tc_clamped(const void* a, const void* w, void* out, int M, in
   return gemm_tc_run(a, w, out, M, N, K, ldo, EPI_CLAMPGLU, bn, splits, partial, status, GluParams{limit, slope}, stream);
 }
 
+// The product with a squared relu and no gate (epilogue 5): out bf16 [M, N] = factor * max(a w^T, 0)^2.
+HK_API int hk_gemm_tc_sqrelu(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int bn, int splits,
+                             float* partial, int* status, float factor, void* stream) {
+  return gemm_tc_run(a, w, out, M, N, K, ldo, EPI_SQRELU, bn, splits, partial, status, GluParams{0.f, factor}, stream);
+}
+
 // Floats of scratch that `hk_gemm_tc` needs for `splits` K slices.
 HK_API long long hk_gemm_tc_partial_floats(int M, int N, int splits) { return (long long)(slice_floats(M, N) * (size_t)splits); }
 
 // The grouped form: a has M rows in tiles of 128 that each belong to one group (groups[tile] = its index, -1: skip the
 // tile), w is [n_groups][N][K] and out has a's rows: out[tile rows] = a[tile rows] w[group]^T.  Epilogue 0 (fp32 store)
-// or 2 (silu(gate) * up, w[group] = [N/2 gate rows | N/2 up rows], out bf16 [M, N/2]).  No K slices.
+// or 2 (silu(gate) * up, w[group] = [N/2 gate rows | N/2 up rows], out bf16 [M, N/2]) or 4 (the same with the clamped
+// activation and its two numbers).  No K slices.
 HK_API int hk_gemm_tc_grouped(const void* a, const void* w, void* out, int M, int N, int K, long long ldo, int epilogue, int bn,
-                              int n_groups, const int* groups, int* status, void* stream) {
+                              int n_groups, const int* groups, int* status, float limit, float slope, void* stream) {
   if (M <= 0 || N <= 0 || n_groups <= 0) return 0;
   if (K <= 0 || (K & 7) || ((uintptr_t)a & 15) || ((uintptr_t)w & 15) || (M % BM) || groups == nullptr) return HK_ERR_UNSUPPORTED;
-  if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU) return HK_ERR_UNSUPPORTED;
+  if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU && epilogue != EPI_CLAMPGLU) return HK_ERR_UNSUPPORTED;
   if (bn < 16 || bn > MAX_BN || (bn & 15)) return HK_ERR_UNSUPPORTED;
   if (IS_GLU(epilogue) && ((N & 1) || (bn & 31))) return HK_ERR_UNSUPPORTED;
   if ((long long)n_groups * N > 0x7fffffffLL) return HK_ERR_UNSUPPORTED;
@@ -624,5 +676,7 @@ HK_API int hk_gemm_tc_grouped(const void* a, const void* w, void* out, int M, in
   if (!make_map(&ma, a, M, K, BM) || !make_map(&mw, w, n_groups * N, K, IS_GLU(epilogue) ? bn / 2 : bn)) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
   if (epilogue == EPI_STORE) return launch<EPI_STORE>(ma, mw, out, M, N, K, ldo, bn, 1, nullptr, status, s, groups);
+  if (epilogue == EPI_CLAMPGLU)
+    return launch<EPI_CLAMPGLU>(ma, mw, out, M, N, K, ldo, bn, 1, nullptr, status, s, groups, GluParams{limit, slope});
   return launch<EPI_SWIGLU>(ma, mw, out, M, N, K, ldo, bn, 1, nullptr, status, s, groups);
 }

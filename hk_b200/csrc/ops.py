@@ -137,8 +137,8 @@ def embedding(table: torch.Tensor, token_ids: torch.Tensor, out: torch.Tensor, s
 
 def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
              rows: Optional[torch.Tensor] = None) -> None:
-    """out[r, :] = x[rows[r] or r, :] * rsqrt(mean(x^2) + eps) * weight  (x, weight float32)."""
-    _need(x, "x", torch.float32, 2)
+    """out[r, :] = x[rows[r] or r, :] * rsqrt(mean(x^2) + eps) * weight  (x, weight float32; x may be a column slice)."""
+    ldx = _cols(x, "x", x.shape[1])
     _need(weight, "weight", torch.float32, 1)
     _need(out, "out", dims=2)
     d = x.shape[1]
@@ -154,7 +154,7 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tenso
             raise KernelError("rms_norm: fewer row indices than output rows")
     lib = build.load("elementwise")
     _check(lib.hk_rms_norm(_ptr(x), _ptr(weight), _ptr(rows), _ptr(out), _dt(out), n_out, d,
-                           ctypes.c_float(eps), _stream()), "rms_norm")
+                           ctypes.c_longlong(ldx), ctypes.c_float(eps), _stream()), "rms_norm")
 
 
 # ---- swiglu ---------------------------------------------------------------------------
@@ -215,6 +215,39 @@ def gemm_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, act
     gu = torch.empty((M, 2 * F), dtype=torch.float32, device=a.device)
     gemm(a, w_gate_up, gu)
     swiglu(gu, out, 0, act, limit, slope)
+
+
+def squared_relu(z: torch.Tensor, out: torch.Tensor, factor: float = 1.0) -> None:
+    """out = factor * max(z, 0)^2 element by element, z float32."""
+    _need(z, "z", torch.float32)
+    _need(out, "out")
+    if z.shape != out.shape:
+        raise KernelError("squared_relu: shapes differ")
+    lib = build.load("elementwise")
+    _check(lib.hk_squared_relu(_ptr(z), _ptr(out), _dt(out), ctypes.c_longlong(z.numel()), ctypes.c_float(factor), _stream()),
+           "squared_relu")
+
+
+def gemm_squared_relu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, factor: float = 1.0) -> None:
+    """out[M, N] = factor * max(a @ w^T, 0)^2 in a's type: in the epilogue of the tensor-core product that takes the shape,
+    else a product to float32 followed by the activation's kernel."""
+    _need(a, "a", dims=2)
+    _need(w, "w", dims=2)
+    _need(out, "out", a.dtype, 2)
+    if w.dtype != a.dtype:                      # weights kept in 32-bit on the bfloat16 path: this product runs in 32-bit
+        wide = torch.empty(out.shape, dtype=w.dtype, device=out.device)
+        gemm_squared_relu(_as_weights(a, w), w, wide, factor)
+        out.copy_(wide)
+        return
+    if a.shape[1] != w.shape[1] or tuple(out.shape) != (a.shape[0], w.shape[0]):
+        raise KernelError("gemm_squared_relu: shapes do not fit")
+    if a.dtype == torch.bfloat16 and _forced["gemm"] != "generic":
+        from . import gemm_fast
+        if gemm_fast.run_squared_relu(a, w, out, factor, _forced["gemm"]):
+            return
+    z = torch.empty(out.shape, dtype=torch.float32, device=a.device)
+    gemm(a, w, z)
+    squared_relu(z, out, factor)
 
 
 # ---- per-head norm + rotation + cache write ---------------------------------------------
@@ -456,10 +489,10 @@ def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, scale: 
                                _stream()), "sigmoid_gate")
 
 
-def latent_prep(proj, q_plain, q_full, c_weight, eps, cos, sin, rotary_dim, pairing, positions, slot_of_token, block_table,
+def latent_prep(q, kv, q_plain, q_full, c_weight, eps, cos, sin, rotary_dim, pairing, positions, slot_of_token, block_table,
                 pages, n_heads, plain_dim, rot_dim, rank, page_tokens, write_kv=True) -> None:
-    """What a token brings to a latent attention, from the fused projection proj float32 [n, >= H*(dn+dr) + r + dr]
-    = [H query heads of (dn plain | dr to rotate) | r compressed dims | dr dims of the shared rotated key | ...]:
+    """What a token brings to a latent attention, from two float32 column slices: q [n, H*(dn+dr)] = H query heads of (dn
+    plain | dr to rotate), and kv [n, r + dr] = r compressed dims, then the dr dims of the shared rotated key:
     q_plain[n, H*dn] takes the queries' plain parts, q_full[n, H*(r+dr)] their rotated parts in its last dr dims per
     head (the first r are left for the absorbed product), and the token's cache row [page, 0, place, r+dr] takes the
     compressed dims RMS-normed with `c_weight` and the rotated key part."""
@@ -470,9 +503,9 @@ def latent_prep(proj, q_plain, q_full, c_weight, eps, cos, sin, rotary_dim, pair
     _need(q_full, "q_full", q_plain.dtype, 2)
     _need(c_weight, "c_weight", torch.float32, 1)
     n = q_plain.shape[0]
-    if not isinstance(proj, torch.Tensor) or not proj.is_cuda or proj.dtype != torch.float32 or proj.dim() != 2 or proj.stride(1) != 1 \
-            or proj.shape[0] != n or proj.shape[1] < H * (dn + dr) + r + dr:
-        raise KernelError("latent_prep: the projection must be float32 [n, >= H*(dn+dr) + r + dr] with unit column stride")
+    ldq, ldkv = _cols(q, "q", H * (dn + dr)), _cols(kv, "kv", r + dr)
+    if q.shape[0] != n or kv.shape[0] != n:
+        raise KernelError("latent_prep: one row of q and kv per token")
     if tuple(q_plain.shape) != (n, H * dn) or tuple(q_full.shape) != (n, H * (r + dr)) or c_weight.shape[0] != r:
         raise KernelError("latent_prep: q_plain, q_full or the norm weight has the wrong shape")
     if rotary_dim > 0:
@@ -489,18 +522,20 @@ def latent_prep(proj, q_plain, q_full, c_weight, eps, cos, sin, rotary_dim, pair
             raise KernelError("latent_prep: cache pages must be [pages, 1, page_tokens, rank + rot_dim]")
     lib = build.load("elementwise")
     _check(lib.hk_latent_prep(
-        _ptr(proj), ctypes.c_longlong(proj.stride(0)), _ptr(q_plain), _ptr(q_full), _dt(q_plain), _ptr(c_weight),
+        _ptr(q), ctypes.c_longlong(ldq), _ptr(kv), ctypes.c_longlong(ldkv), _ptr(q_plain), _ptr(q_full), _dt(q_plain), _ptr(c_weight),
         ctypes.c_float(eps), _ptr(cos if rotary_dim > 0 else None), _ptr(sin if rotary_dim > 0 else None), int(rotary_dim),
         PAIRINGS[pairing], _ptr(positions), _ptr(slot_of_token), _ptr(block_table if write_kv else None),
         int(block_table.shape[1]) if write_kv else 0, _ptr(pages if write_kv else None), n, H, dn, dr, r, int(page_tokens),
         1 if write_kv else 0, _stream()), "latent_prep")
 
 
-def gemm_heads(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_heads: int, gate: Optional[torch.Tensor] = None) -> None:
+def gemm_heads(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_heads: int, gate: Optional[torch.Tensor] = None,
+               gate_scale: float = 1.0, gate_per_head: bool = False) -> None:
     """One small product per head: out[t, h, :N] = a[t, h, :K] @ w[h]^T for w [H, N, K].  `a` and `out` are 3-D views
     [n, H, K] and [n, H, N] with any row and head strides and unit stride along the last dimension (so either may be
     a slice of wider heads).  out takes a's type or float32.  `gate` (a float32 column slice [n, H * N] of a projection's
-    output): the result is multiplied by sigmoid(gate), head h reading columns h * N .. of it."""
+    output): the result is multiplied by gate_scale * sigmoid(gate), head h reading columns h * N .. of it; with
+    `gate_per_head` the gate is a slice [n, H] and head h's result is multiplied by one number."""
     H = n_heads
     for name, t in (("a", a), ("out", out)):
         if not isinstance(t, torch.Tensor) or not t.is_cuda or t.dim() != 3 or t.stride(2) != 1 or t.shape[1] != H:
@@ -512,21 +547,23 @@ def gemm_heads(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_heads: int
         raise KernelError("gemm_heads: shapes do not fit")
     gate_ld = 0
     if gate is not None:
-        gate_ld = _cols(gate, "gate", H * N)
+        gate_ld = _cols(gate, "gate", H if gate_per_head else H * N)
         if gate.shape[0] != n:
             raise KernelError("gemm_heads: one row of gate logits per row")
     if a.dtype == torch.bfloat16 and _forced["gemm"] != "generic":
         lib = build.load("gemm_heads")
         code = lib.hk_gemm_heads_mma(_ptr(a), _ptr(w), _ptr(out), _dt(out), n, N, K, H, ctypes.c_longlong(a.stride(0)),
                                      ctypes.c_longlong(a.stride(1)), ctypes.c_longlong(out.stride(0)),
-                                     ctypes.c_longlong(out.stride(1)), _ptr(gate), ctypes.c_longlong(gate_ld), _stream())
+                                     ctypes.c_longlong(out.stride(1)), _ptr(gate), ctypes.c_longlong(gate_ld),
+                                     1 if gate_per_head else 0, ctypes.c_float(gate_scale), _stream())
         if code != _ERR_UNSUPPORTED:
             _check(code, "gemm_heads (mma)")
             return
     lib = build.load("gemm_generic")
     _check(lib.hk_gemm_heads(_ptr(a), _ptr(w), _dt(a), _ptr(out), _dt(out), n, N, K, H, ctypes.c_longlong(a.stride(0)),
                              ctypes.c_longlong(a.stride(1)), ctypes.c_longlong(out.stride(0)), ctypes.c_longlong(out.stride(1)),
-                             _ptr(gate), ctypes.c_longlong(gate_ld), _stream()), "gemm_heads")
+                             _ptr(gate), ctypes.c_longlong(gate_ld), 1 if gate_per_head else 0, ctypes.c_float(gate_scale),
+                             _stream()), "gemm_heads")
 
 
 # ---- sampling -------------------------------------------------------------------------
@@ -609,9 +646,10 @@ def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor)
            "polynorm")
 
 
-def _cols(x: torch.Tensor, name: str, width: int) -> int:
-    """Checks a float32 column slice [n, width] of a row-major matrix; returns its row stride."""
-    if not isinstance(x, torch.Tensor) or not x.is_cuda or x.dtype != torch.float32 or x.dim() != 2:
+def _cols(x: torch.Tensor, name: str, width: int, any_type: bool = False) -> int:
+    """Checks a float32 (with `any_type` also bfloat16) column slice [n, width] of a row-major matrix; returns its row stride."""
+    if not isinstance(x, torch.Tensor) or not x.is_cuda or x.dim() != 2 \
+            or (x.dtype != torch.float32 and not (any_type and x.dtype == torch.bfloat16)):
         raise KernelError(f"{name} must be a float32 CUDA matrix")
     if x.shape[1] != width or x.stride(1) != 1:
         raise KernelError(f"{name} must be [n, {width}] with unit column stride")
@@ -697,13 +735,17 @@ def mingru_scan(proj, z_bias, x_bias, segments, state, out) -> None:
                               int(segments.shape[0]), _ptr(state), _ptr(out), _dt(out), W, _stream()), "mingru_scan")
 
 
-def short_conv(x, weight, segments, tail, out, act: str = "silu") -> None:
-    """out[t, c] = act(sum_j weight[c, j] * x[t - (taps - 1) + j, c]) over the rows of every segment (the last column
-    of `weight` is the current token's); act 'silu' or 'none'.  Rows before a segment's first come from `tail` float32 [slots, taps - 1, C],
+def short_conv(x, weight, segments, tail, out, act: str = "silu", bias=None) -> None:
+    """out[t, c] = act(bias[c] + sum_j weight[c, j] * x[t - (taps - 1) + j, c]) over the rows of every segment (the last
+    column of `weight` is the current token's); act 'silu' or 'none', bias float32 [C] or None.  Rows before a segment's first come from `tail` float32 [slots, taps - 1, C],
     the request's last taps - 1 inputs (zero at its start), which is moved on (with one tap: one row that is left alone).
-    x and out: float32 column slices [n, C]."""
+    x: a float32 column slice [n, C]; out: a column slice [n, C] of float32 or bfloat16."""
     C = int(weight.shape[0])
-    ldx, ldy = _cols(x, "x", C), _cols(out, "out", C)
+    ldx, ldy = _cols(x, "x", C), _cols(out, "out", C, any_type=True)
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != C:
+            raise KernelError("short_conv: one bias per channel")
     _need(weight, "weight", torch.float32, 2)
     _need(segments, "segments", torch.int32, 2)
     _need(tail, "tail", torch.float32, 3)
@@ -711,9 +753,9 @@ def short_conv(x, weight, segments, tail, out, act: str = "silu") -> None:
     if x.shape[0] != out.shape[0] or tuple(tail.shape[1:]) != (max(taps - 1, 1), C) or segments.shape[1] != 3 or taps < 1 \
             or act not in ("silu", "none"):
         raise KernelError("short_conv: shapes do not fit")
-    lib = build.load("recurrent")
-    _check(lib.hk_short_conv(_ptr(x), ctypes.c_longlong(ldx), _ptr(weight), _ptr(segments), int(segments.shape[0]), int(x.shape[0]),
-                             _ptr(tail), _ptr(out), ctypes.c_longlong(ldy), C, taps, 1 if act == "silu" else 0, _stream()),
+    lib = build.load("short_conv")
+    _check(lib.hk_short_conv(_ptr(x), ctypes.c_longlong(ldx), _ptr(weight), _ptr(bias), _ptr(segments), int(segments.shape[0]),
+                             int(x.shape[0]), _ptr(tail), _ptr(out), _dt(out), ctypes.c_longlong(ldy), C, taps, 1 if act == "silu" else 0, _stream()),
            "short_conv")
 
 
@@ -779,6 +821,47 @@ def retention_scan(q, k, v, cos, sin, rotary_dim: int, positions, decay, segment
                                  _ptr(sin if rotary_dim > 0 else None), int(rotary_dim), _ptr(positions), _ptr(decay), _ptr(segments),
                                  int(segments.shape[0]), n, _ptr(rec), _ptr(state), _ptr(out), H, dk, dv, ctypes.c_float(k_scale),
                                  _stream()), "retention_scan", launches=2)
+
+
+def state_space_scan(xbc, dt_logit, dt_bias, a_log, skip, segments, state, out, n_heads: int, n_groups: int, state_dim: int,
+                     value_dim: int) -> None:
+    """The state-space recurrence over the rows of every segment, per head, S = state[slot, head] float32 (stored [dv, N]):
+        dt = softplus(dt_logit + dt_bias);  S <- exp(-exp(a_log) dt) S + dt B x^T;  out = S^T C + skip x
+    xbc [n, H*dv + 2*G*N] (a column slice, float32 or bfloat16) = [x | B | C]; head h reads group h // (H/G) of B and C;
+    dt_logit a float32 column slice [n, H]; dt_bias, a_log, skip float32 [H]; out float32 [n, H*dv]."""
+    H, G, N, dv = n_heads, n_groups, state_dim, value_dim
+    ldx = _cols(xbc, "xbc", H * dv + 2 * G * N, any_type=True)
+    ldt = _cols(dt_logit, "dt_logit", H)
+    for name, t in (("dt_bias", dt_bias), ("a_log", a_log), ("skip", skip)):
+        _need(t, name, torch.float32, 1)
+        if t.shape[0] != H:
+            raise KernelError(f"state_space_scan: {name} must have one entry per head")
+    _need(segments, "segments", torch.int32, 2)
+    _need(state, "state", torch.float32, 4)
+    _need(out, "out", torch.float32, 2)
+    n = xbc.shape[0]
+    if H % G or tuple(state.shape[1:]) != (H, dv, N) or tuple(out.shape) != (n, H * dv) or dt_logit.shape[0] != n \
+            or segments.shape[1] != 3:
+        raise KernelError("state_space_scan: shapes do not fit")
+    lib = build.load("state_space")
+    _check(lib.hk_state_space_walk(_ptr(xbc), _dt(xbc), ctypes.c_longlong(ldx), _ptr(dt_logit), ctypes.c_longlong(ldt), _ptr(dt_bias),
+                                   _ptr(a_log), _ptr(skip), _ptr(segments), int(segments.shape[0]), n, _ptr(state), _ptr(out), H, G, N,
+                                   dv, _stream()), "state_space_scan")
+
+
+def gated_part_norm(y, z, weight, eps: float, out, parts: int) -> None:
+    """u = y * silu(z); out = every one of `parts` equal parts of a row of u over sqrt(mean(u^2) + eps) of that part, times
+    weight.  y float32 [n, W], z a float32 column slice [n, W], weight float32 [W]."""
+    _need(y, "y", torch.float32, 2)
+    n, W = y.shape
+    ldz = _cols(z, "z", W)
+    _need(weight, "weight", torch.float32, 1)
+    _need(out, "out", dims=2)
+    if tuple(out.shape) != (n, W) or z.shape[0] != n or weight.shape[0] != W or W % parts:
+        raise KernelError("gated_part_norm: shapes do not fit")
+    lib = build.load("state_space")
+    _check(lib.hk_gated_part_norm(_ptr(y), _ptr(z), ctypes.c_longlong(ldz), _ptr(weight), _ptr(out), _dt(out), n, W, int(parts),
+                                  ctypes.c_float(eps), _stream()), "gated_part_norm")
 
 
 def mlstm_padded(value_dim: int) -> int:
@@ -897,6 +980,9 @@ def route_tile_rows() -> int:
     return int(build.load("routed").hk_route_tile_rows())
 
 
+ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_all": 2}
+
+
 def route_topk(x, w_router, ids, weights, scores: str = "softmax", correction=None, groups: int = 0, keep: int = 0,
                scale: float = 1.0, norm_eps: float = 0.0, extra_out=None) -> None:
     """Per row of x [n, d]: the `top` = ids.shape[1] largest of the E float32 router logits x . w_router[e]
@@ -905,7 +991,8 @@ def route_topk(x, w_router, ids, weights, scores: str = "softmax", correction=No
     None), among the experts of the best `keep` of `groups` equal groups of neighbours when groups > 0 (a group's score: the
     sum of its two largest choice scores; the others count as minus infinity); weights = s / (sum of the chosen s +
     norm_eps) * scale.  `extra_out` float32 [n, X]: w_router has X more rows behind the experts', and the sigmoids of their
-    logits are written there."""
+    logits are written there.  scores 'softmax_all': s = softmax over all E logits, the choice is made on s + correction,
+    weights = s * scale (not renormalised)."""
     _need(x, "x", dims=2)
     _need(w_router, "w_router", torch.float32, 2)
     _need(ids, "ids", torch.int32, 2)
@@ -918,7 +1005,7 @@ def route_topk(x, w_router, ids, weights, scores: str = "softmax", correction=No
         if extra_out.shape[0] != n:
             raise KernelError("route_topk: one row of extra_out per row of x")
     E = int(w_router.shape[0]) - extra
-    if w_router.shape[1] != d or ids.shape[0] != n or ids.shape != weights.shape or scores not in ("softmax", "sigmoid") or E < 1:
+    if w_router.shape[1] != d or ids.shape[0] != n or ids.shape != weights.shape or scores not in ROUTE_SCORES or E < 1:
         raise KernelError("route_topk: shapes do not fit")
     if correction is not None:
         _need(correction, "correction", torch.float32, 1)
@@ -926,13 +1013,13 @@ def route_topk(x, w_router, ids, weights, scores: str = "softmax", correction=No
             raise KernelError("route_topk: one correction per expert")
     lib = build.load("routed")
     _check(lib.hk_route_topk(_ptr(x), _dt(x), _ptr(w_router), _ptr(ids), _ptr(weights), n, d, E, ids.shape[1],
-                             1 if scores == "sigmoid" else 0, _ptr(correction), int(groups), int(keep), ctypes.c_float(scale),
+                             ROUTE_SCORES[scores], _ptr(correction), int(groups), int(keep), ctypes.c_float(scale),
                              ctypes.c_float(norm_eps), extra, _ptr(extra_out), _stream()), "route_topk")
 
 
 def route_sort(ids, n_experts: int, offsets, perm, inv, tiles) -> None:
     """Lays the (row, choice) pairs out by expert: offsets int32 [E+1], perm [pairs] (sorted place -> pair), inv [pairs]
-    (pair -> sorted place), tiles int32 [max_tiles, 2] = (expert, first sorted place) of every tile of
+    (pair -> sorted place, -1 for an id of n_experts or more: an identity), tiles int32 [max_tiles, 2] = (expert, first sorted place) of every tile of
     `route_tile_rows()` rows, -1 for unused tiles."""
     for name, t in (("ids", ids), ("offsets", offsets), ("perm", perm), ("inv", inv), ("tiles", tiles)):
         _need(t, name, torch.int32)
@@ -944,10 +1031,13 @@ def route_sort(ids, n_experts: int, offsets, perm, inv, tiles) -> None:
                              _stream()), "route_sort")
 
 
-def grouped_gemm(a, w, out, tiles, offsets, perm, top: int, gather: bool, gated: bool) -> None:
+def grouped_gemm(a, w, out, tiles, offsets, perm, top: int, gather: bool, gated: bool, act: str = "silu", limit: float = 0.0,
+                 slope: float = 1.0) -> None:
     """A product per expert over the sorted rows.  w [E, N, K] (gated: [E, 2N, K] = N gate rows then N up rows);
     row p of the product reads a[perm[p] // top] (gather) or a[p]; out[p, :N] = a . w[e]^T in float32, or
-    silu(gate) * up in a's type when gated."""
+    silu(gate) * up (or the clamped form of `swiglu`) in a's type when gated."""
+    if act not in ("silu", "swish_clamped"):
+        raise KernelError(f"grouped_gemm: activation {act!r} is neither 'silu' nor 'swish_clamped'")
     _need(a, "a", dims=2)
     _need(w, "w", a.dtype, 3)
     _need(out, "out", dims=2)
@@ -957,12 +1047,14 @@ def grouped_gemm(a, w, out, tiles, offsets, perm, top: int, gather: bool, gated:
         raise KernelError("grouped_gemm: shapes or types do not fit")
     lib = build.load("routed")
     _check(lib.hk_grouped_gemm(_ptr(a), _ptr(w), _dt(a), _ptr(out), _ptr(tiles), tiles.shape[0], _ptr(offsets), _ptr(perm),
-                               int(top), 1 if gather else 0, N, K, 1 if gated else 0, _stream()), "grouped_gemm")
+                               int(top), 1 if gather else 0, N, K, 1 if gated else 0, 1 if act == "swish_clamped" else 0,
+                               ctypes.c_float(limit), ctypes.c_float(slope), _stream()), "grouped_gemm")
 
 
-def route_combine(ys, inv, weights, y, accumulate: bool = False, shared=None, shared_gate=None) -> None:
-    """y[t, :] (+)= sum_k weights[t, k] * ys[inv[t, k], :], the choices in their order (all float32); with `shared`
-    (float32 [n, d]) also + shared_gate[t] * shared[t, :] (shared_gate float32 [n] or [n, 1]; None: 1)."""
+def route_combine(ys, inv, weights, y, accumulate: bool = False, shared=None, shared_gate=None, x=None, factor: float = 1.0) -> None:
+    """y[t, :] (+)= factor * (sum_k weights[t, k] * ys[inv[t, k], :]), the choices in their order (all float32); with
+    `shared` (float32 [n, d]) also + shared_gate[t] * shared[t, :] inside the brackets (shared_gate float32 [n] or [n, 1];
+    None: 1).  A choice with inv[t, k] = -1 is an identity: it takes x[t, :] (x [n, d], float32 or bfloat16)."""
     _need(ys, "ys", torch.float32, 2)
     _need(inv, "inv", torch.int32)
     _need(weights, "weights", torch.float32, 2)
@@ -975,9 +1067,14 @@ def route_combine(ys, inv, weights, y, accumulate: bool = False, shared=None, sh
         if shared.shape != y.shape or (shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.numel() != n
                                                                     or not shared_gate.is_contiguous())):
             raise KernelError("route_combine: the shared result must be [n, d] and its gate [n]")
+    if x is not None:
+        _need(x, "x", dims=2)
+        if x.shape != y.shape:
+            raise KernelError("route_combine: x must be [n, d]")
     lib = build.load("routed")
     _check(lib.hk_route_combine(_ptr(ys), _ptr(inv), _ptr(weights), _ptr(y), n, y.shape[1], top, 1 if accumulate else 0,
-                                _ptr(shared), _ptr(shared_gate if shared is not None else None), _stream()), "route_combine")
+                                _ptr(shared), _ptr(shared_gate if shared is not None else None), _ptr(x),
+                                _dt(x) if x is not None else F32, ctypes.c_float(factor), _stream()), "route_combine")
 
 
 def route_sort_padded(ids, n_experts: int, pad: int, perm, inv, groups) -> None:
@@ -1005,9 +1102,9 @@ def route_gather(x, perm, top: int, xs) -> None:
     _check(lib.hk_route_gather(_ptr(x), _ptr(perm), int(top), _ptr(xs), xs.shape[0], xs.shape[1], _stream()), "route_gather")
 
 
-def grouped_gemm_tc(a, w, out, groups, gated: bool) -> bool:
+def grouped_gemm_tc(a, w, out, groups, gated: bool, act: str = "silu", limit: float = 0.0, slope: float = 1.0) -> bool:
     """The grouped product on the tcgen05 kernel: a bf16 [M, K] in tiles of 128 rows, tile t belonging to expert groups[t]
-    (-1: skipped); w bf16 [E, N, K] (gated: [E, 2N, K]); out float32 [M, N], or bf16 silu(gate) * up when gated.  False when
+    (-1: skipped); w bf16 [E, N, K] (gated: [E, 2N, K]); out float32 [M, N], or bf16 silu(gate) * up (or the clamped form) when gated.  False when
     the kernel refuses the shape."""
     from . import gemm_fast
-    return gemm_fast.run_grouped(a, w, out, groups, gated)
+    return gemm_fast.run_grouped(a, w, out, groups, gated, GLU_ACTS[act], limit, slope)

@@ -484,82 +484,6 @@ HK_API int hk_mingru_scan(const float* proj, long long ld, const float* z_bias, 
   return HK_ERR_UNSUPPORTED;
 }
 
-// ------------------------------------------------------------------ short causal convolution per channel
-// y[t, c] = act(sum_j w[c, j] * x[t - (taps - 1) + j, c]) over the rows of every segment, with act = silu (1) or the
-// identity (0): the last column of w is the current token's.  The inputs before a segment's first row come from the request's tail
-// (state [slots, taps - 1, C], the last taps - 1 inputs of the request, zero at its start), which the same call
-// moves on.  x and y are column slices [n, C] of wider float32 matrices.  A thread owns one channel of one chunk
-// of a segment's tokens; the threads of the first chunk read the old tail before they write the new one, and
-// nobody else touches it.
-#define SC_TOKENS 32
-#define SC_GROUP 8
-#define SC_MAX_TAPS 16
-
-// The thread walks its tokens in groups of SC_GROUP: the group's inputs are loaded at once (each input is read once; the
-// taps - 1 before them stay in registers from the group before), then the group's outputs are summed, oldest tap first.
-__global__ void __launch_bounds__(128)
-short_conv_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w, const int* __restrict__ segs,
-                  float* __restrict__ tail, float* __restrict__ y, long long ldy, int C, int taps, int act) {
-  const int seg = blockIdx.x;
-  const int c = blockIdx.y * blockDim.x + threadIdx.x;
-  const int slot = segs[seg * 3], row0 = segs[seg * 3 + 1], count = segs[seg * 3 + 2];
-  const int t0 = blockIdx.z * SC_TOKENS;
-  if (c >= C || t0 >= count) return;
-  const int back = taps - 1;
-  float* tl = tail + (size_t)slot * back * C + c;
-  auto input = [&](int r) -> float {            // the request's input r rows from the segment's first (r may be negative)
-    return r >= 0 ? x[(size_t)(row0 + r) * ldx + c] : tl[(size_t)(back + r) * C];
-  };
-  float wr[SC_MAX_TAPS];                        // wr[s]: the weight of the input s tokens back
-  float hist[SC_MAX_TAPS];                      // hist[s], s >= 1: the input s tokens before the group's first
-#pragma unroll
-  for (int s = 0; s < SC_MAX_TAPS; ++s) {
-    wr[s] = s <= back ? w[(size_t)c * taps + back - s] : 0.f;
-    hist[s] = (s >= 1 && s <= back) ? input(t0 - s) : 0.f;
-  }
-  const int t1 = min(count, t0 + SC_TOKENS);
-  for (int tg = t0; tg < t1; tg += SC_GROUP) {
-    float nw[SC_GROUP];
-#pragma unroll
-    for (int u = 0; u < SC_GROUP; ++u) nw[u] = tg + u < t1 ? x[(size_t)(row0 + tg + u) * ldx + c] : 0.f;
-    float acc[SC_GROUP];
-#pragma unroll
-    for (int u = 0; u < SC_GROUP; ++u) acc[u] = 0.f;
-#pragma unroll
-    for (int s = SC_MAX_TAPS - 1; s >= 0; --s) {
-      if (s <= back) {
-#pragma unroll
-        for (int u = 0; u < SC_GROUP; ++u) acc[u] = fmaf(wr[s], u >= s ? nw[u - s] : hist[s - u], acc[u]);
-      }
-    }
-#pragma unroll
-    for (int u = 0; u < SC_GROUP; ++u)
-      if (tg + u < t1) y[(size_t)(row0 + tg + u) * ldy + c] = act ? acc[u] / (1.0f + expf(-acc[u])) : acc[u];
-    float next[SC_MAX_TAPS];
-#pragma unroll
-    for (int s = 1; s < SC_MAX_TAPS; ++s) next[s] = s <= SC_GROUP ? nw[SC_GROUP - s] : hist[s - SC_GROUP];
-#pragma unroll
-    for (int s = 1; s < SC_MAX_TAPS; ++s) hist[s] = next[s];
-  }
-  if (blockIdx.z == 0 && back > 0) {
-    float keep[SC_MAX_TAPS];
-#pragma unroll
-    for (int j = 0; j < SC_MAX_TAPS; ++j)
-      if (j < back) keep[j] = input(count - back + j);
-#pragma unroll
-    for (int j = 0; j < SC_MAX_TAPS; ++j)
-      if (j < back) tl[(size_t)j * C] = keep[j];
-  }
-}
-
-HK_API int hk_short_conv(const float* x, long long ldx, const float* w, const int* segs, int n_seg, int n_rows, float* tail,
-                         float* y, long long ldy, int C, int taps, int act, void* stream) {
-  if (n_seg <= 0 || n_rows <= 0 || C <= 0) return 0;
-  if (taps < 1 || taps > SC_MAX_TAPS || act < 0 || act > 1) return HK_ERR_UNSUPPORTED;
-  dim3 grid((unsigned)n_seg, (unsigned)((C + 127) / 128), (unsigned)((n_rows + SC_TOKENS - 1) / SC_TOKENS));
-  return hk_launch(short_conv_kernel, grid, dim3(128), 0, (cudaStream_t)stream, x, ldx, w, segs, tail, y, ldy, C, taps, act);
-}
-
 // ------------------------------------------------------------------ gated delta rule
 // Per head a matrix state S [dk, dv] and per token a scalar decay g and a scalar write strength beta:
 //     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q

@@ -8,14 +8,19 @@
 //               expert by itself: s = sigmoid(logit); the choice is made on s + correction (a float per expert),
 //               optionally among the experts of the best `keep` of `groups` equal groups of neighbours (a
 //               group's score: the sum of its two largest choice scores), and the weights are the chosen
-//               experts' s over their sum (+ norm_eps), times a factor.  The router's matrix may carry further
+//               experts' s over their sum (+ norm_eps), times a factor.  A third mode takes s = softmax over all the
+//               logits, chooses on s + correction and gives the chosen s themselves (times a factor) as weights.
+//               The router's matrix may carry further
 //               rows behind the experts' (`extra`): their logits' sigmoids are handed out per token (a gate
 //               of a sublayer that every token uses).
+//               The last outputs of the router may stand for no feed-forward at all (identities: such a choice gives
+//               back the token's vector); the sort leaves their pairs out and the combine adds the vector itself.
 //   2. sort:    one CTA counts the (token, choice) pairs per expert, lays the experts' rows out one after
 //               the other (`perm`: sorted place -> pair, `inv`: pair -> sorted place) and cuts every
 //               expert's rows into tiles of RT_BM rows (`tiles`: expert and first row, -1 for unused).
 //   3. experts: a grouped product over those tiles: tile rows are gathered through `perm`, the weights are
-//               the tile's expert's; first gate and up with silu(gate) * up in the epilogue, then down.
+//               the tile's expert's; first gate and up with silu(gate) * up (or the clamped
+//               activation) in the epilogue, then down.
 //               A row's result does not depend on its place in a tile: every output element is one chain of
 //               k = 0..K-1 (the FMA kernel) or a fixed tree (the tensor-core kernel).
 //   4. combine: y[t] = sum over the token's choices, in the order of the choices, of weight * expert output.
@@ -30,10 +35,10 @@
 // ------------------------------------------------------------------------------------ 1. route
 #define RK_WARPS 8
 struct RouteOpts {
-  int mode;                  // 0: softmax over the chosen logits; 1: sigmoid scores
-  const float* correction;   // mode 1: added to the scores for the choice alone (null: nothing)
+  int mode;                  // 0: softmax over the chosen logits; 1: sigmoid scores; 2: softmax over all logits, not renormalised
+  const float* correction;   // modes 1 and 2: added to the scores for the choice alone (null: nothing)
   int groups, keep;          // mode 1: the choice is made inside the best `keep` of `groups` groups (groups 0: everywhere)
-  float scale, norm_eps;     // mode 1: weights = s / (sum s + norm_eps) * scale
+  float scale, norm_eps;     // mode 1: weights = s / (sum s + norm_eps) * scale; mode 2: weights = s * scale
   int extra;                 // rows of w behind the E experts' rows
   float* extra_out;          // [n, extra]: the sigmoids of those rows' logits
 };
@@ -91,6 +96,22 @@ route_topk_kernel(const T* __restrict__ x, const float* __restrict__ w, int* __r
   __syncthreads();
   if (wid != 0) return;
   E = n_experts;
+  if (opt.mode == 2) {
+    float top_z = -CUDART_INF_F, sum = 0.f;
+    for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, z[e]);
+    top_z = warp_max(top_z);
+    for (int e = lane; e < E; e += 32) {
+      score[e] = expf(z[e] - top_z);
+      sum += score[e];
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      const float sc = score[e] / sum;
+      score[e] = sc;
+      z[e] = opt.correction != nullptr ? sc + opt.correction[e] : sc;
+    }
+    __syncwarp();
+  }
   if (opt.mode == 1) {
     for (int e = lane; e < E; e += 32) {
       const float sc = 1.0f / (1.0f + expf(-z[e]));
@@ -165,8 +186,8 @@ route_topk_kernel(const T* __restrict__ x, const float* __restrict__ w, int* __r
       }
     }
     if (k == 0) first = best;
-    // mode 0: the first chosen logit is the largest; mode 1: the expert's own score, without the correction
-    const float p = opt.mode == 1 ? (bi < E ? score[bi] : 0.f) : expf(best - first);
+    // mode 0: the first chosen logit is the largest; modes 1 and 2: the expert's own score, without the correction
+    const float p = opt.mode != 0 ? (bi < E ? score[bi] : 0.f) : expf(best - first);
     total += p;
     if (lane == (k & 31)) {                    // lane k keeps choice k (top <= 32)
       mine = p;
@@ -177,7 +198,7 @@ route_topk_kernel(const T* __restrict__ x, const float* __restrict__ w, int* __r
   }
   if (lane < top) {
     ids[(size_t)t * top + lane] = mine_id < E ? mine_id : 0;
-    weights[(size_t)t * top + lane] = opt.mode == 1 ? mine / (total + opt.norm_eps) * opt.scale : mine / total;
+    weights[(size_t)t * top + lane] = opt.mode == 1 ? mine / (total + opt.norm_eps) * opt.scale : opt.mode == 2 ? mine * opt.scale : mine / total;
   }
 }
 
@@ -185,8 +206,9 @@ HK_API int hk_route_topk(const void* x, int dtype, const float* w, int* ids, flo
                          const float* correction, int groups, int keep, float scale, float norm_eps, int extra, float* extra_out,
                          void* stream) {
   if (n <= 0) return 0;
-  if (E < 1 || top < 1 || top > E || top > 32 || E > 2048 || mode < 0 || mode > 1 || extra < 0 || extra > 64) return HK_ERR_UNSUPPORTED;
+  if (E < 1 || top < 1 || top > E || top > 32 || E > 2048 || mode < 0 || mode > 2 || extra < 0 || extra > 64) return HK_ERR_UNSUPPORTED;
   if (mode == 0 && (correction != nullptr || groups != 0 || extra != 0)) return HK_ERR_UNSUPPORTED;
+  if (mode == 2 && (groups != 0 || extra != 0)) return HK_ERR_UNSUPPORTED;
   if (groups < 0 || (groups > 0 && (E % groups || keep < 1 || keep > groups)) || (extra > 0 && extra_out == nullptr)) return HK_ERR_UNSUPPORTED;
   const RouteOpts opt = {mode, correction, groups, keep, scale, norm_eps, extra, extra_out};
   const size_t smem = ((size_t)(RK_WARPS + 1) * (E + extra) + E + 2 * groups) * sizeof(float);
@@ -206,7 +228,8 @@ HK_API int hk_route_topk(const void* x, int dtype, const float* w, int* ids, flo
 }
 
 // ------------------------------------------------------------------------------------ 2. sort
-// offsets[E + 1], perm[pairs], inv[pairs], tiles[max_tiles][2].
+// offsets[E + 1], perm[pairs], inv[pairs], tiles[max_tiles][2].  A pair whose id is E or more (an identity) has no sorted
+// place: its inv is -1.
 __global__ void __launch_bounds__(1024)
 route_sort_kernel(const int* __restrict__ ids, int pairs, int E, int bm, int* __restrict__ offsets, int* __restrict__ perm,
                   int* __restrict__ inv, int* __restrict__ tiles, int max_tiles) {
@@ -215,7 +238,8 @@ route_sort_kernel(const int* __restrict__ ids, int pairs, int E, int bm, int* __
   int* cursor = smi + E;
   for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < pairs; p += blockDim.x) atomicAdd(&counts[ids[p]], 1);
+  for (int p = threadIdx.x; p < pairs; p += blockDim.x)
+    if (ids[p] < E) atomicAdd(&counts[ids[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0, tile = 0;
@@ -237,6 +261,10 @@ route_sort_kernel(const int* __restrict__ ids, int pairs, int E, int bm, int* __
   }
   __syncthreads();
   for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+    if (ids[p] >= E) {
+      inv[p] = -1;
+      continue;
+    }
     const int at = atomicAdd(&cursor[ids[p]], 1);
     perm[at] = p;
     inv[p] = at;
@@ -265,7 +293,8 @@ route_sort_padded_kernel(const int* __restrict__ ids, int pairs, int E, int pad,
   for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
   for (int p = threadIdx.x; p < m_max; p += blockDim.x) perm[p] = -1;
   __syncthreads();
-  for (int p = threadIdx.x; p < pairs; p += blockDim.x) atomicAdd(&counts[ids[p]], 1);
+  for (int p = threadIdx.x; p < pairs; p += blockDim.x)
+    if (ids[p] < E) atomicAdd(&counts[ids[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0;
@@ -279,6 +308,10 @@ route_sort_padded_kernel(const int* __restrict__ ids, int pairs, int E, int pad,
   }
   __syncthreads();
   for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+    if (ids[p] >= E) {
+      inv[p] = -1;
+      continue;
+    }
     const int at = atomicAdd(&cursor[ids[p]], 1);
     perm[at] = p;
     inv[p] = at;
@@ -311,13 +344,26 @@ HK_API int hk_route_gather(const void* x, const int* perm, int top, void* xs, in
 
 
 // ------------------------------------------------------------------------------------ 3. experts
+struct GluAct {
+  int clamped;               // 0: silu(gate) * up; 1: g sigmoid(slope g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+  float limit, slope;
+};
+__device__ __forceinline__ float glu_value(float g, float u, GluAct act) {
+  if (act.clamped) {
+    g = fminf(g, act.limit);
+    u = fminf(fmaxf(u, -act.limit), act.limit);
+    return g / (1.0f + expf(-act.slope * g)) * (u + 1.0f);
+  }
+  return g / (1.0f + expf(-g)) * u;
+}
+
 // out rows are sorted places.  GATED: w is [E][2N][K] = N gate rows then N up rows per expert, out[p, n] (type TO) =
-// silu(gate) * up.  Otherwise w is [E][N][K] and out[p, n] (float) = a[p] . w[e][n].  `gather`: row p of `a` is row
+// the gated activation `act` of the two.  Otherwise w is [E][N][K] and out[p, n] (float) = a[p] . w[e][n].  `gather`: row p of `a` is row
 // perm[p] / top of the tensor (the token's vector); else row p.
 template <typename T, typename TO, bool GATED>
 __global__ void __launch_bounds__(256)
 grouped_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, TO* __restrict__ out, const int* __restrict__ tiles,
-                    const int* __restrict__ offsets, const int* __restrict__ perm, int top, int gather, int N, int K) {
+                    const int* __restrict__ offsets, const int* __restrict__ perm, int top, int gather, int N, int K, GluAct act) {
   __shared__ float As[RT_BK][RT_BM + 4];
   __shared__ float Ws[GATED ? 2 : 1][RT_BK][RT_BN + 4];
   __shared__ int rows[RT_BM];
@@ -381,8 +427,7 @@ grouped_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, TO* __rest
       if (gn >= N) continue;
       float val = acc[0][i][j];
       if (GATED) {
-        const float u = acc[GATED ? 1 : 0][i][j];
-        val = val / (1.0f + expf(-val)) * u;
+        val = glu_value(val, acc[GATED ? 1 : 0][i][j], act);
       }
       out[(size_t)p * N + gn] = from_f32<TO>(val);
     }
@@ -391,7 +436,7 @@ grouped_gemm_kernel(const T* __restrict__ a, const T* __restrict__ w, TO* __rest
 
 // The same on the tensor cores (bf16 operands, fp32 accumulation; K a multiple of 8): a CTA takes a tile of RT_BM
 // sorted rows and 128 weight rows: plain, 128 output columns; gated, 64 gate rows and the 64 up rows that match
-// them, so that silu(gate) * up is taken in the epilogue.  Operands come through a three-stage cp.async ring in
+// them, so that the gated activation is taken in the epilogue.  Operands come through a three-stage cp.async ring in
 // slices of 32 k (A rows gathered through `rows`), fragments by ldmatrix, products by mma.sync m16n8k16: eight
 // warps as 2 (rows) x 4 (columns), a warp 32 rows x 32 weight rows.  An output element's sum runs over k in an
 // order that does not depend on the row's place in its tile, so a token's result does not depend on the batch.
@@ -419,7 +464,7 @@ __device__ __forceinline__ void gm_mma(float* c, const uint32_t* a, uint32_t b0,
 template <bool GATED, int GM_STAGES>
 __global__ void __launch_bounds__(256)
 grouped_gemm_mma_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, void* __restrict__ out_, const int* __restrict__ tiles,
-                        const int* __restrict__ offsets, const int* __restrict__ perm, int top, int gather, int N, int K) {
+                        const int* __restrict__ offsets, const int* __restrict__ perm, int top, int gather, int N, int K, GluAct act) {
   extern __shared__ __align__(16) uint8_t gm_smem[];
   typedef bf16 (*ATile)[RT_BM][GM_LD];
   typedef bf16 (*WTile)[GM_BN][GM_LD];
@@ -513,7 +558,7 @@ grouped_gemm_mma_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, 
             const int gn = n0 + wc * 16 + nt * 8 + t2 + c;
             if (gn >= N) continue;
             const float gate = acc[mt][nt][half * 2 + c], up = acc[mt][nt + 2][half * 2 + c];
-            out[(size_t)p * N + gn] = __float2bfloat16_rn(gate / (1.0f + expf(-gate)) * up);
+            out[(size_t)p * N + gn] = __float2bfloat16_rn(glu_value(gate, up, act));
           }
       } else {
         float* out = reinterpret_cast<float*>(out_);
@@ -530,72 +575,87 @@ grouped_gemm_mma_kernel(const bf16* __restrict__ a, const bf16* __restrict__ w, 
 
 template <bool GATED, int STAGES>
 static int gm_launch(const void* a, const void* w, void* out, const int* tiles, int max_tiles, const int* offsets, const int* perm,
-                     int top, int gather, int N, int K, cudaStream_t s) {
+                     int top, int gather, int N, int K, GluAct act, cudaStream_t s) {
   const size_t smem = sizeof(bf16) * STAGES * (RT_BM + GM_BN) * GM_LD;
   static HkSmemCache cache;
   if (int e = hk_allow_smem(grouped_gemm_mma_kernel<GATED, STAGES>, smem, cache)) return e;
   dim3 grid((unsigned)((N + (GATED ? 63 : GM_BN - 1)) / (GATED ? 64 : GM_BN)), (unsigned)max_tiles);
   return hk_launch(grouped_gemm_mma_kernel<GATED, STAGES>, grid, dim3(256), smem, s, (const bf16*)a, (const bf16*)w, out, tiles, offsets,
-                   perm, top, gather, N, K);
+                   perm, top, gather, N, K, act);
 }
 
 HK_API int hk_grouped_gemm(const void* a, const void* w, int dtype, void* out, const int* tiles, int max_tiles, const int* offsets,
-                           const int* perm, int top, int gather, int N, int K, int gated, void* stream) {
+                           const int* perm, int top, int gather, int N, int K, int gated, int clamped, float limit, float slope,
+                           void* stream) {
   if (max_tiles <= 0 || N <= 0) return 0;
   if (max_tiles > 65535) return HK_ERR_UNSUPPORTED;
+  const GluAct act = {clamped, limit, slope};
   dim3 grid((unsigned)((N + RT_BN - 1) / RT_BN), (unsigned)max_tiles);
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == HK_F32) {
     if (gated)
       return hk_launch(grouped_gemm_kernel<float, float, true>, grid, dim3(256), 0, s, (const float*)a, (const float*)w, (float*)out,
-                       tiles, offsets, perm, top, gather, N, K);
+                       tiles, offsets, perm, top, gather, N, K, act);
     return hk_launch(grouped_gemm_kernel<float, float, false>, grid, dim3(256), 0, s, (const float*)a, (const float*)w, (float*)out,
-                     tiles, offsets, perm, top, gather, N, K);
+                     tiles, offsets, perm, top, gather, N, K, act);
   }
   if (dtype == HK_BF16 && (K & 7) == 0 && ((((uintptr_t)a | (uintptr_t)w) & 15) == 0)) {
     // few rows (decode steps): the products are bound by the experts' weight bytes, and a ring of six slices keeps more of
     // them on their way (width 4,096, 128 pairs: 88 and 45 us against 97 and 57 with three); many rows: three slices leave
     // room for four CTAs an SM (4,096 pairs: 546 and 297 us against 653 and 307 with six)
     const bool deep = max_tiles <= 40;       // tiles = pairs / 64 + experts: a few hundred pairs at most
-    if (gated) return deep ? gm_launch<true, 6>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, s)
-                           : gm_launch<true, 3>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, s);
-    return deep ? gm_launch<false, 6>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, s)
-                : gm_launch<false, 3>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, s);
+    if (gated) return deep ? gm_launch<true, 6>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, act, s)
+                           : gm_launch<true, 3>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, act, s);
+    return deep ? gm_launch<false, 6>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, act, s)
+                : gm_launch<false, 3>(a, w, out, tiles, max_tiles, offsets, perm, top, gather, N, K, act, s);
   }
   if (dtype == HK_BF16) {
     if (gated)
       return hk_launch(grouped_gemm_kernel<bf16, bf16, true>, grid, dim3(256), 0, s, (const bf16*)a, (const bf16*)w, (bf16*)out, tiles,
-                       offsets, perm, top, gather, N, K);
+                       offsets, perm, top, gather, N, K, act);
     return hk_launch(grouped_gemm_kernel<bf16, float, false>, grid, dim3(256), 0, s, (const bf16*)a, (const bf16*)w, (float*)out, tiles,
-                     offsets, perm, top, gather, N, K);
+                     offsets, perm, top, gather, N, K, act);
   }
   return HK_ERR_UNSUPPORTED;
 }
 
 // ------------------------------------------------------------------------------------ 4. combine
-// y[t, :] (= or +=) sum_k weights[t, k] * ys[inv[t * top + k], :] (+ shared_gate[t] * shared[t, :], the result of a
-// sublayer that every token uses, when `shared` is given; a null gate counts as 1)
+// y[t, :] (= or +=) factor * (sum_k weights[t, k] * ys[inv[t * top + k], :] (+ shared_gate[t] * shared[t, :], the result of
+// a sublayer that every token uses, when `shared` is given; a null gate counts as 1)).  A choice whose inv is negative is
+// an identity: it adds weights[t, k] * x[t, :], the token's own vector.
+template <typename T>
 __global__ void route_combine_kernel(const float* __restrict__ ys, const int* __restrict__ inv, const float* __restrict__ weights,
                                      float* __restrict__ y, int d, int top, int accumulate, const float* __restrict__ shared,
-                                     const float* __restrict__ shared_gate) {
+                                     const float* __restrict__ shared_gate, const T* __restrict__ x, float factor) {
   const int t = blockIdx.x;
   const float sg = shared != nullptr ? (shared_gate != nullptr ? shared_gate[t] : 1.0f) : 0.f;
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < d; i += gridDim.y * blockDim.x) {
     float acc = 0.f;
-    for (int k = 0; k < top; ++k) acc = fmaf(weights[(size_t)t * top + k], ys[(size_t)inv[(size_t)t * top + k] * d + i], acc);
+    for (int k = 0; k < top; ++k) {
+      const int at = inv[(size_t)t * top + k];
+      const float v = at >= 0 ? ys[(size_t)at * d + i] : x != nullptr ? to_f32<T>(x[(size_t)t * d + i]) : 0.f;
+      acc = fmaf(weights[(size_t)t * top + k], v, acc);
+    }
     if (shared != nullptr) acc = fmaf(sg, shared[(size_t)t * d + i], acc);
     float* o = y + (size_t)t * d + i;
-    *o = accumulate ? *o + acc : acc;
+    *o = accumulate ? fmaf(factor, acc, *o) : factor * acc;
   }
 }
 
 HK_API int hk_route_combine(const float* ys, const int* inv, const float* weights, float* y, int n, int d, int top, int accumulate,
-                            const float* shared, const float* shared_gate, void* stream) {
+                            const float* shared, const float* shared_gate, const void* x, int x_dtype, float factor, void* stream) {
   if (n <= 0) return 0;
   // a block per token; where the tokens alone do not fill the SMs (decode steps) a token's columns are spread over blocks
   const int threads = d >= 1024 ? 256 : 128;
   int split = 1;
   while (split < 16 && (long long)n * split < 2 * 148 && split * threads < d) split <<= 1;
-  return hk_launch(route_combine_kernel, dim3((unsigned)n, (unsigned)split), dim3(threads), 0, (cudaStream_t)stream, ys, inv, weights,
-                   y, d, top, accumulate, shared, shared_gate);
+  const dim3 grid((unsigned)n, (unsigned)split);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (x_dtype == HK_F32)
+    return hk_launch(route_combine_kernel<float>, grid, dim3(threads), 0, s, ys, inv, weights, y, d, top, accumulate, shared, shared_gate,
+                     (const float*)x, factor);
+  if (x_dtype == HK_BF16)
+    return hk_launch(route_combine_kernel<bf16>, grid, dim3(threads), 0, s, ys, inv, weights, y, d, top, accumulate, shared, shared_gate,
+                     (const bf16*)x, factor);
+  return HK_ERR_UNSUPPORTED;
 }

@@ -109,6 +109,18 @@ class Precision:
         raise ValueError(f"unknown parameter kind '{kind}'")
 
 
+def stacked_rows(matrices, multiple: int = 1) -> torch.Tensor:
+    """Several weights [out, in] over the same input as one, so that one product gives all of their results side by side.
+    Where one of them is kept in 32-bit, all are.  `multiple`: zero rows fill the result up to a multiple of it (results
+    whose rows stay aligned for wide loads whatever the sizes are)."""
+    wide = torch.float32 if any(t.dtype == torch.float32 for t in matrices) else matrices[0].dtype
+    rows = [t.to(wide) for t in matrices]
+    spare = -sum(int(t.shape[0]) for t in rows) % multiple
+    if spare:
+        rows.append(torch.zeros((spare, rows[0].shape[1]), dtype=wide, device=rows[0].device))
+    return torch.cat(rows, dim=0).contiguous()
+
+
 class Part:
     """Base of all parts.  Sub-parts are found through `children()`.
 

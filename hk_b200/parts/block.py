@@ -10,7 +10,7 @@ from __future__ import annotations
 import torch
 
 from .base import Part, register_part
-from .parallel import mixer_cache_specs, mixer_caches
+from .parallel import mixer_cache_specs, mixer_caches, takes_scale
 
 
 class PreNormBlock(Part):
@@ -122,3 +122,40 @@ class PostNormBlock(Part):
 
 
 register_part("block", "post_norm", PostNormBlock)
+
+
+class ParallelBlock(Part):
+    """A layer with one norm whose output both sublayers read:
+        x <- x + scale * (mixer(N(x)) + ffn(N(x)))
+    Where both sublayers can carry a factor on their result (a settable `out_scale`), they are given `scale` when the block
+    is made and add their output projections straight onto the float32 residual stream; otherwise they fill a float32
+    buffer that one kernel adds onto the stream times `scale`.  The feed-forward may be absent."""
+    graph_safe = True   # reads the batch from device tensors only
+
+    def __init__(self, norm, mixer, feed_forward=None, scale: float = 1.0):
+        self.norm, self.mixer, self.feed_forward, self.scale = norm, mixer, feed_forward, float(scale)
+        parts = [p for p in (mixer, feed_forward) if p is not None]
+        self._carried = self.scale == 1.0 or all(takes_scale(p) for p in parts)
+        if self._carried and self.scale != 1.0:
+            for p in parts:
+                p.out_scale = self.scale * p.out_scale
+
+    def children(self):
+        return tuple(p for p in (self.norm, self.mixer, self.feed_forward) if p is not None)
+
+    def cache_specs(self):
+        return mixer_cache_specs(self.mixer)
+
+    def forward(self, residual: torch.Tensor, ctx, caches, write_cache: bool = True) -> None:
+        from ..csrc import ops
+        xb = torch.empty(residual.shape, dtype=ctx.precision.compute, device=residual.device)
+        self.norm.forward(residual, xb)
+        y = residual if self._carried else torch.empty_like(residual)
+        self.mixer.forward(xb, y, ctx, mixer_caches(self.mixer, caches), write_cache, accumulate=self._carried)
+        if self.feed_forward is not None:
+            self.feed_forward.forward(xb, y, ctx, accumulate=True)
+        if not self._carried:
+            ops.scaled_sum(residual, y, self.scale)
+
+
+register_part("block", "parallel", ParallelBlock)

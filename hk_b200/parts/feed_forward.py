@@ -58,6 +58,30 @@ class SwiGLUFeedForward(Part):
 register_part("feed_forward", "swiglu", SwiGLUFeedForward)
 
 
+class SquaredReLUFeedForward(Part):
+    """residual += out_scale * W_down max(W_up xb, 0)^2, no gate and no biases; the activation (with the factor) runs in the
+    epilogue of the up product where a tensor-core product takes it."""
+    graph_safe = True   # reads the batch from device tensors only
+
+    def __init__(self, hidden: int, intermediate: int, prefix: str, names=None, out_scale: float = 1.0):
+        self.hidden, self.F, self.prefix, self.out_scale = hidden, intermediate, prefix, float(out_scale)
+        self.names = {"up": "up", "down": "down"}
+        self.names.update(names or {})
+        self.w_up = self.w_down = None
+
+    def own_param_specs(self) -> Dict[str, ParamSpec]:
+        p, nm = self.prefix, self.names
+        return {p + nm["up"]: ParamSpec((self.F, self.hidden), MATRIX), p + nm["down"]: ParamSpec((self.hidden, self.F), MATRIX)}
+
+    def own_bind(self, tensors, precision: Precision) -> None:
+        self.w_up, self.w_down = tensors[self.prefix + self.names["up"]], tensors[self.prefix + self.names["down"]]
+
+    def forward(self, xb: torch.Tensor, residual: torch.Tensor, ctx, accumulate: bool = True) -> None:
+        h = torch.empty((xb.shape[0], self.F), dtype=xb.dtype, device=xb.device)
+        ops.gemm_squared_relu(xb, self.w_up, h, self.out_scale)
+        ops.gemm(h, self.w_down, residual, accumulate=accumulate)
+
+
 class PolyNormFeedForward(Part):
     """residual += W_down act(W_up xb) with the polynomial activation
         act(z) = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3,   N(v) = v / sqrt(mean(v^2) + eps) over a token's F values,
@@ -106,7 +130,13 @@ class RoutedFeedForward(Part):
     choice scores; the experts of the other groups count as minus infinity), and the weights are the chosen experts' s over
     their sum + `norm_eps`, times `weight_scale`.  `shared`: one more feed-forward part that every token uses; its result is
     added to the experts' sum, times sigmoid(W_sg xb) (one number per token, tensor `shared_gate` [1, d], whose product
-    rides along with the router's in 32-bit) when `shared_gated` is set."""
+    rides along with the router's in 32-bit) when `shared_gated` is set.
+
+    `scores="softmax_all"` is a third router: s = softmax(z) over all of its outputs, the choice is made on s + correction,
+    and the weights are the chosen s themselves (times `weight_scale`).  `identity`: the router has that many further
+    outputs behind the experts' which stand for no feed-forward: such a choice gives back xb itself, times its weight.
+    `act`, `limit`, `slope` are the experts' gated activation (silu, or the clamped form of `SwiGLUFeedForward`);
+    `out_scale` is a factor on the whole result."""
     graph_safe = True   # reads the batch from device tensors only; launches depend on the row count alone
     kernel_libraries = ("routed",)
     route_log = None    # a list, when someone wants to see the choices: every eager forward appends a copy of its
@@ -114,11 +144,16 @@ class RoutedFeedForward(Part):
 
     def __init__(self, hidden: int, intermediate: int, n_experts: int, top: int, prefix: str, names=None,
                  scores: str = "softmax", correction: bool = False, groups: int = 0, keep: int = 0, weight_scale: float = 1.0,
-                 norm_eps: float = 0.0, shared=None, shared_gated: bool = False):
-        if not 1 <= top <= n_experts or top > 32:
-            raise ValueError(f"top = {top} must be in 1..min(experts, 32) (experts = {n_experts})")
-        if scores not in ("softmax", "sigmoid"):
-            raise ValueError(f"scores '{scores}' is neither 'softmax' nor 'sigmoid'")
+                 norm_eps: float = 0.0, shared=None, shared_gated: bool = False, identity: int = 0, act: str = "silu",
+                 limit: float = 0.0, slope: float = 1.0, out_scale: float = 1.0):
+        if identity < 0 or not 1 <= top <= n_experts + identity or top > 32:
+            raise ValueError(f"top = {top} must be in 1..min(experts, 32) (experts = {n_experts}, identities = {identity})")
+        if scores not in ops.ROUTE_SCORES:
+            raise ValueError(f"scores '{scores}' is not one of {', '.join(ops.ROUTE_SCORES)}")
+        if scores == "softmax_all" and (groups or shared_gated):
+            raise ValueError("groups and a gated shared part belong to scores='sigmoid'")
+        if act not in ("silu", "swish_clamped") or (act == "swish_clamped" and not limit > 0):
+            raise ValueError("the experts' activation is 'silu', or 'swish_clamped' with a positive limit")
         if scores == "softmax" and (correction or groups or weight_scale != 1.0 or shared_gated):
             raise ValueError("a correction, groups, a factor on the weights and a gated shared part belong to scores='sigmoid'")
         if groups and (n_experts % groups or not 1 <= keep <= groups):
@@ -129,6 +164,8 @@ class RoutedFeedForward(Part):
         self.scores, self.correction, self.groups, self.keep = scores, bool(correction), int(groups), int(keep)
         self.weight_scale, self.norm_eps = float(weight_scale), float(norm_eps)
         self.shared, self.shared_gated = shared, bool(shared_gated)
+        self.identity, self.act, self.limit, self.slope = int(identity), act, float(limit), float(slope)
+        self.out_scale = float(out_scale)
         self.names = {"router": "router", "expert": "e{}.", "gate": "gate", "up": "up", "down": "down",
                       "correction": "correction", "shared_gate": "shared.sg"}
         self.names.update(names or {})
@@ -141,9 +178,10 @@ class RoutedFeedForward(Part):
         return self.prefix + self.names["expert"].format(e) + self.names[which]
 
     def own_param_specs(self) -> Dict[str, ParamSpec]:
-        specs = {self.prefix + self.names["router"]: ParamSpec((self.E, self.hidden), MATRIX)}
+        outputs = self.E + self.identity
+        specs = {self.prefix + self.names["router"]: ParamSpec((outputs, self.hidden), MATRIX)}
         if self.correction:
-            specs[self.prefix + self.names["correction"]] = ParamSpec((self.E,), VECTOR)
+            specs[self.prefix + self.names["correction"]] = ParamSpec((outputs,), VECTOR)
         if self.shared_gated:
             specs[self.prefix + self.names["shared_gate"]] = ParamSpec((1, self.hidden), MATRIX)
         for e in range(self.E):
@@ -180,13 +218,17 @@ class RoutedFeedForward(Part):
         xs = torch.empty((m_max, self.hidden), dtype=xb.dtype, device=dev)
         ops.route_gather(xb, perm, self.top, xs)
         h = torch.empty((m_max, self.F), dtype=xb.dtype, device=dev)
-        if not ops.grouped_gemm_tc(xs, self.w_gate_up, h, groups, gated=True):
+        if not ops.grouped_gemm_tc(xs, self.w_gate_up, h, groups, gated=True, act=self.act, limit=self.limit, slope=self.slope):
             return False
         ys = torch.empty((m_max, self.hidden), dtype=torch.float32, device=dev)
         if not ops.grouped_gemm_tc(h, self.w_down, ys, groups, gated=False):
             return False
-        ops.route_combine(ys, inv, weights, residual, accumulate=accumulate, shared=shared_y, shared_gate=shared_gate)
+        self._combine(ys, inv, weights, xb, residual, accumulate, shared_y, shared_gate)
         return True
+
+    def _combine(self, ys, inv, weights, xb, residual, accumulate: bool, shared_y, shared_gate) -> None:
+        ops.route_combine(ys, inv, weights, residual, accumulate=accumulate, shared=shared_y, shared_gate=shared_gate,
+                          x=xb if self.identity else None, factor=self.out_scale)
 
     def forward(self, xb: torch.Tensor, residual: torch.Tensor, ctx, accumulate: bool = True) -> None:
         n, dev = xb.shape[0], xb.device
@@ -212,11 +254,13 @@ class RoutedFeedForward(Part):
         tiles = torch.empty((max_tiles, 2), dtype=torch.int32, device=dev)
         ops.route_sort(ids, self.E, offsets, perm, inv, tiles)
         h = torch.empty((pairs, self.F), dtype=xb.dtype, device=dev)
-        ops.grouped_gemm(xb, self.w_gate_up, h, tiles, offsets, perm, self.top, gather=True, gated=True)
+        ops.grouped_gemm(xb, self.w_gate_up, h, tiles, offsets, perm, self.top, gather=True, gated=True, act=self.act,
+                         limit=self.limit, slope=self.slope)
         ys = torch.empty((pairs, self.hidden), dtype=torch.float32, device=dev)
         ops.grouped_gemm(h, self.w_down, ys, tiles, offsets, perm, self.top, gather=False, gated=False)
-        ops.route_combine(ys, inv, weights, residual, accumulate=accumulate, shared=shared_y, shared_gate=shared_gate)
+        self._combine(ys, inv, weights, xb, residual, accumulate, shared_y, shared_gate)
 
 
+register_part("feed_forward", "squared_relu", SquaredReLUFeedForward)
 register_part("feed_forward", "polynorm", PolyNormFeedForward)
 register_part("feed_forward", "routed_swiglu", RoutedFeedForward)

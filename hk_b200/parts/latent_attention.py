@@ -12,7 +12,10 @@ per head), the attention runs as H query heads over one shared key/value head wh
 [c | k_rot] and whose value is the row's first kv_rank dims, and W_uv,h is applied to the attention's result
 (sum_j p_j c_j).  A decode step therefore reads kv_rank + rot_dim numbers per cached token, whatever the number of
 heads.  Sizes, the norm's eps, the position encoding (its pairing, scaling and magnitude), the scale, a window and
-the output gate are parameters; `names` renames the tensors (keys q, dkv, dkv_norm, uk, uv, gate, o).
+the output gate are parameters; `names` renames the tensors (keys q, dkv, dkv_norm, uk, uv, gate, o, dq, dq_norm, uq).
+  `q_rank`: the queries come through a latent of their own, q = W_uq (rms(W_dq x) * weight), instead of W_q x;
+  `gate="head"`: one gate number per head (tensor [n_heads, hidden]) instead of one per output of a head;
+  `out_scale` is a factor on the mixer's result that the gate carries.
 """
 from __future__ import annotations
 
@@ -21,7 +24,7 @@ from typing import Dict, Optional
 import torch
 
 from ..csrc import ops
-from .base import KVCacheSpec, MATRIX, VECTOR, ParamSpec, Part, Precision, register_part
+from .base import KVCacheSpec, MATRIX, VECTOR, ParamSpec, Part, Precision, register_part, stacked_rows
 from .position import RotaryEmbedding
 
 
@@ -29,8 +32,9 @@ class LatentAttention(Part):
     graph_safe = True   # reads the batch from device tensors only
 
     def __init__(self, hidden: int, n_heads: int, plain_dim: int, rot_dim: int, v_head_dim: int, kv_rank: int, prefix: str,
-                 norm_eps: float, scale: float, position: Optional[RotaryEmbedding] = None, gate: bool = False,
-                 window: Optional[int] = None, names: Optional[Dict[str, str]] = None):
+                 norm_eps: float, scale: float, position: Optional[RotaryEmbedding] = None, gate=False,
+                 window: Optional[int] = None, names: Optional[Dict[str, str]] = None, q_rank: Optional[int] = None,
+                 out_scale: float = 1.0):
         if min(n_heads, plain_dim, v_head_dim, kv_rank) < 1 or rot_dim < 0:
             raise ValueError("heads, plain_dim, v_head_dim and kv_rank must be positive, rot_dim not negative")
         if kv_rank + rot_dim > 640:
@@ -40,9 +44,16 @@ class LatentAttention(Part):
         self.hidden, self.H, self.dn, self.dr, self.vd, self.r = hidden, n_heads, plain_dim, rot_dim, v_head_dim, kv_rank
         self.prefix, self.norm_eps, self.scale = prefix, float(norm_eps), float(scale)
         self.position, self.gate, self.window = position, bool(gate), window
-        self.names = {"q": "q", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "gate": "g", "o": "o"}
+        self.gate_per_head = gate == "head"
+        if q_rank is not None and q_rank < 1:
+            raise ValueError("q_rank must be positive (or absent)")
+        if out_scale != 1.0 and not gate:
+            raise ValueError("out_scale rides on the output gate: it needs a gate")
+        self.q_rank, self.out_scale = q_rank, float(out_scale)
+        self.names = {"q": "q", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "gate": "g", "o": "o",
+                      "dq": "dq", "dq_norm": "dq.norm", "uq": "uq"}
         self.names.update(names or {})
-        self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.c_norm = None
+        self.w_in = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = self.c_norm = self.q_norm = None
         self._tables_key = None        # set at bind: the flash kernels' work items, when they take a row of this size
         self._sm_count = 0
         self._wide = False             # set at bind: the row is too wide for the flash kernels, the latent kernel takes it
@@ -83,15 +94,20 @@ class LatentAttention(Part):
     def own_param_specs(self) -> Dict[str, ParamSpec]:
         p, nm, H, d = self.prefix, self.names, self.H, self.hidden
         specs = {
-            p + nm["q"]: ParamSpec((H * (self.dn + self.dr), d), MATRIX),
             p + nm["dkv"]: ParamSpec((self.r + self.dr, d), MATRIX),
             p + nm["dkv_norm"]: ParamSpec((self.r,), VECTOR, "one_plus_normal"),
             p + nm["uk"]: ParamSpec((H * self.dn, self.r), MATRIX),
             p + nm["uv"]: ParamSpec((H * self.vd, self.r), MATRIX),
             p + nm["o"]: ParamSpec((d, H * self.vd), MATRIX),
         }
+        if self.q_rank is None:
+            specs[p + nm["q"]] = ParamSpec((H * (self.dn + self.dr), d), MATRIX)
+        else:
+            specs[p + nm["dq"]] = ParamSpec((self.q_rank, d), MATRIX)
+            specs[p + nm["dq_norm"]] = ParamSpec((self.q_rank,), VECTOR, "one_plus_normal")
+            specs[p + nm["uq"]] = ParamSpec((H * (self.dn + self.dr), self.q_rank), MATRIX)
         if self.gate:
-            specs[p + nm["gate"]] = ParamSpec((H * self.vd, d), MATRIX)
+            specs[p + nm["gate"]] = ParamSpec((H if self.gate_per_head else H * self.vd, d), MATRIX)
         return specs
 
     def cache_spec(self):
@@ -100,9 +116,11 @@ class LatentAttention(Part):
 
     def own_bind(self, tensors, precision: Precision) -> None:
         p, nm, H = self.prefix, self.names, self.H
-        mats = [tensors[p + nm["q"]], tensors[p + nm["dkv"]]] + ([tensors[p + nm["gate"]]] if self.gate else [])
-        wide = torch.float32 if any(t.dtype == torch.float32 for t in mats) else mats[0].dtype
-        self.w_in = torch.cat([t.to(wide) for t in mats], dim=0).contiguous()       # one product: q, compressed row, gate
+        # one product: q (or its latent), compressed row, gate
+        self.w_in = stacked_rows([tensors[p + nm["q" if self.q_rank is None else "dq"]], tensors[p + nm["dkv"]]]
+                                 + ([tensors[p + nm["gate"]]] if self.gate else []), multiple=8 if self.q_rank is not None else 1)
+        if self.q_rank is not None:
+            self.w_uq, self.q_norm = tensors[p + nm["uq"]], tensors[p + nm["dq_norm"]]
         dt = precision.compute
         # q_lat,h = W_uk,h^T q_plain,h: as a product with weights [out = kv_rank, in = plain_dim] per head
         self.w_uk_t = tensors[p + nm["uk"]].to(dt).view(H, self.dn, self.r).transpose(1, 2).contiguous()
@@ -149,6 +167,15 @@ class LatentAttention(Part):
         H, dn, dr, r, vd = self.H, self.dn, self.dr, self.r, self.vd
         proj = torch.empty((n, self.w_in.shape[0]), dtype=torch.float32, device=dev)
         ops.gemm(xb, self.w_in, proj)
+        if self.q_rank is None:
+            at = H * (dn + dr)
+            q = proj[:, :at]
+        else:
+            at = self.q_rank
+            c_q = torch.empty((n, at), dtype=dt, device=dev)
+            ops.rms_norm(proj[:, :at], self.q_norm, self.norm_eps, c_q)
+            q = torch.empty((n, H * (dn + dr)), dtype=torch.float32, device=dev)
+            ops.gemm(c_q, self.w_uq, q)
         q_plain = torch.empty((n, H * dn), dtype=dt, device=dev)
         q_full = torch.empty((n, H * (r + dr)), dtype=dt, device=dev)
         cos = sin = None
@@ -156,14 +183,15 @@ class LatentAttention(Part):
         if self.position is not None:
             cos, sin, rot = self.position.tables()
             pairing = self.position.pairing
-        ops.latent_prep(proj, q_plain, q_full, self.c_norm, self.norm_eps, cos, sin, rot, pairing, ctx.positions,
+        ops.latent_prep(q, proj[:, at:at + r + dr], q_plain, q_full, self.c_norm, self.norm_eps, cos, sin, rot, pairing, ctx.positions,
                         ctx.slot_of_token, cache.block_table, cache.k_pages, H, dn, dr, r, cache.page_tokens,
                         write_kv=write_cache)
         ops.gemm_heads(q_plain.view(n, H, dn), self.w_uk_t, q_full.view(n, H, r + dr)[:, :, :r], H)
         lat = self._attend(q_full, ctx, cache)                  # [n, H, r]: sum_j p_j c_j per head
         att = torch.empty((n, H * vd), dtype=dt, device=dev)
         # the values' up-projection per head, with the output gate in its epilogue
-        ops.gemm_heads(lat, self.w_uv, att.view(n, H, vd), H, gate=proj[:, H * (dn + dr) + r + dr:] if self.gate else None)
+        gate = proj[:, at + r + dr:at + r + dr + (H if self.gate_per_head else H * vd)] if self.gate else None
+        ops.gemm_heads(lat, self.w_uv, att.view(n, H, vd), H, gate=gate, gate_scale=self.out_scale, gate_per_head=self.gate_per_head)
         ops.gemm(att, self.w_o, residual, accumulate=accumulate)
 
 

@@ -26,8 +26,8 @@ def mixer_caches(mixer, caches):
     return list(caches) if hasattr(mixer, "cache_specs") else caches[0]
 
 
-def _takes_scale(mixer) -> bool:
-    """Whether the mixer carries a factor on its result by itself (set before its tensors are bound)."""
+def takes_scale(mixer) -> bool:
+    """Whether a mixer or feed-forward carries a factor on its result by itself (set before its tensors are bound)."""
     return hasattr(mixer, "out_scale") and bool(getattr(mixer, "gate", True))      # an attention carries it on its gate
 
 
@@ -38,7 +38,7 @@ class ParallelMixer(Part):
         self.left, self.right = left, right
         self.left_scale, self.right_scale = float(left_scale), float(right_scale)
         self._n_left = len(mixer_cache_specs(left))
-        self._carried = all(_takes_scale(m) for m in (left, right))
+        self._carried = all(takes_scale(m) for m in (left, right))
         if self._carried:
             left.out_scale, right.out_scale = self.left_scale, self.right_scale
 

@@ -43,8 +43,14 @@ denominator):
       y = W_o ((o / rms(o) per head) * silu(W_g h))
   `decay` (one number per head) and `k_scale` (key_dim^(-1/2) by default) are parameters.
 
+`StateSpace` (Mamba-2; per head a matrix state S [state_dim, value_dim], zero at the start; head h reads B and C of group
+h // (n_heads / n_groups)):
+      [z | x | B | C | dt] = W_in h;   x, B, C <- silu(conv(x, B, C) + bias)          a short causal convolution per channel
+      dt <- softplus(dt + dt_bias);   S <- exp(-exp(A_log) dt) S + dt B x^T;   o = S^T C + D x
+      y = W_o (N(o * silu(z)) * norm_weight),   N over each of `norm_groups` equal parts of the n_heads * value_dim numbers
+
 `ShortConvolution` is the causal convolution over a request's last `taps` rows per channel as a part of its own (tensors
-[channels, taps] by group of channels, an optional silu, the request's last taps - 1 inputs as its state), for mixers
+[channels, taps] by group of channels, an optional bias and silu, the request's last taps - 1 inputs as its state), for mixers
 other than the gated delta rule that put one behind their projections.
 
 A mixer with several caches says so with `cache_specs()` and is handed the list.
@@ -58,7 +64,7 @@ import numpy as np
 import torch
 
 from ..csrc import ops
-from .base import MATRIX, VECTOR, ParamSpec, Part, Precision, StateSpec, StepTables, register_part
+from .base import MATRIX, VECTOR, ParamSpec, Part, Precision, StateSpec, StepTables, register_part, stacked_rows
 
 SEGMENTS_KEY = ("request_segments",)
 
@@ -186,6 +192,8 @@ class MinGRU(_SegmentScan):
 
 
 class GatedDeltaRule(_SegmentScan):
+    kernel_libraries = ("recurrent", "short_conv")
+
     def __init__(self, hidden: int, n_heads: int, kv_heads: int, key_dim: int, value_dim: int, taps: int, prefix: str,
                  norm_eps: float, unit_eps: float = 1e-6, q_scale: Optional[float] = None, out_scale: float = 1.0,
                  names: Optional[Dict[str, str]] = None):
@@ -309,18 +317,24 @@ class Retention(_SegmentScan):
 
 
 class ShortConvolution(_SegmentScan):
-    """y[t, c] = act(sum_j w[c, j] x[t - (taps - 1) + j, c]) over a request's rows, zeros before its start.  `groups`:
-    (tensor name, channels) in the order of the channels; the tensors [channels, taps] are laid side by side at binding."""
+    """y[t, c] = act(b[c] + sum_j w[c, j] x[t - (taps - 1) + j, c]) over a request's rows, zeros before its start.  `groups`:
+    (tensor name, channels) in the order of the channels; the tensors [channels, taps] are laid side by side at binding.
+    `bias`: every tensor has a bias [channels] beside it, whose name ends in ".b"; without, b = 0."""
+    kernel_libraries = ("short_conv",)
 
-    def __init__(self, groups, taps: int, act: str = "none"):
+    def __init__(self, groups, taps: int, act: str = "none", bias: bool = False):
         if taps < 1 or act not in ("none", "silu"):
             raise ValueError("the short convolution needs at least one tap, and act 'none' or 'silu'")
         self.groups, self.taps, self.act = [(str(nm), int(c)) for nm, c in groups], int(taps), act
         self.channels = sum(c for _, c in self.groups)
-        self.weight = None
+        self.has_bias = bool(bias)
+        self.weight = self.bias = None
 
     def own_param_specs(self) -> Dict[str, ParamSpec]:
-        return {nm: ParamSpec((c, self.taps), VECTOR) for nm, c in self.groups}
+        specs = {nm: ParamSpec((c, self.taps), VECTOR) for nm, c in self.groups}
+        if self.has_bias:
+            specs.update({nm + ".b": ParamSpec((c,), VECTOR) for nm, c in self.groups})
+        return specs
 
     def cache_spec(self):
         # one tap keeps no inputs; its tail is a row that nobody reads (a state of no size has no slot to live in)
@@ -328,10 +342,79 @@ class ShortConvolution(_SegmentScan):
 
     def own_bind(self, tensors, precision: Precision) -> None:
         self.weight = torch.cat([tensors[nm] for nm, _ in self.groups], dim=0).contiguous()
+        if self.has_bias:
+            self.bias = torch.cat([tensors[nm + ".b"] for nm, _ in self.groups], dim=0).contiguous()
 
     def forward(self, x: torch.Tensor, ctx, cache, out: torch.Tensor) -> None:
-        """x and out: float32 column slices [n, channels]; `cache`: the state of `cache_spec()`."""
-        ops.short_conv(x, self.weight, self._segments(ctx), cache.state, out, act=self.act)
+        """x: a float32 column slice [n, channels]; out: one of float32 or the compute type; `cache`: the state of
+        `cache_spec()`."""
+        ops.short_conv(x, self.weight, self._segments(ctx), cache.state, out, act=self.act, bias=self.bias)
+
+
+class StateSpace(_SegmentScan):
+    """`out_scale` is a factor on the mixer's result (carried by the norm's weight).  The input projection's one tensor is
+    the product's weight as it is, filled up to a multiple of 8 rows."""
+    kernel_libraries = ("state_space",)
+
+    def __init__(self, hidden: int, n_heads: int, value_dim: int, state_dim: int, n_groups: int, taps: int, prefix: str,
+                 norm_eps: float, norm_groups: int = 1, out_scale: float = 1.0, names: Optional[Dict[str, str]] = None):
+        if n_heads % n_groups:
+            raise ValueError(f"{n_heads} heads are not a multiple of {n_groups} groups")
+        if (n_heads * value_dim) % norm_groups:
+            raise ValueError(f"{n_heads} heads of {value_dim} do not form {norm_groups} equal parts for the norm")
+        self.hidden, self.H, self.dv, self.N, self.G = hidden, n_heads, value_dim, state_dim, n_groups
+        self.prefix, self.norm_eps, self.norm_groups, self.out_scale = prefix, float(norm_eps), int(norm_groups), float(out_scale)
+        self.names = {"in": "in", "conv": "conv", "dt_bias": "dt_bias", "a_log": "A_log", "skip": "D", "norm": "norm", "o": "o"}
+        self.names.update(names or {})
+        self.conv = ShortConvolution([(prefix + self.names["conv"], self.channels)], taps, act="silu", bias=True)
+        self.w_in = self.w_o = self.dt_bias = self.a_log = self.skip = self.norm_weight = None
+
+    @property
+    def inner(self) -> int:
+        return self.H * self.dv
+
+    @property
+    def channels(self) -> int:
+        """What passes the convolution: x, B and C."""
+        return self.inner + 2 * self.G * self.N
+
+    def children(self):
+        return (self.conv,)
+
+    def own_param_specs(self) -> Dict[str, ParamSpec]:
+        p, nm, d, H = self.prefix, self.names, self.hidden, self.H
+        return {
+            p + nm["in"]: ParamSpec((self.inner + self.channels + H, d), MATRIX),
+            p + nm["dt_bias"]: ParamSpec((H,), VECTOR), p + nm["a_log"]: ParamSpec((H,), VECTOR), p + nm["skip"]: ParamSpec((H,), VECTOR),
+            p + nm["norm"]: ParamSpec((self.inner,), VECTOR, "one_plus_normal"), p + nm["o"]: ParamSpec((d, self.inner), MATRIX),
+        }
+
+    def cache_specs(self):
+        return [StateSpec((self.H, self.dv, self.N), torch.float32), self.conv.cache_spec()]
+
+    def own_bind(self, tensors, precision: Precision) -> None:
+        p, nm = self.prefix, self.names
+        self.w_in = stacked_rows([tensors[p + nm["in"]]], multiple=8)
+        self.w_o = tensors[p + nm["o"]]
+        self.dt_bias, self.a_log, self.skip = tensors[p + nm["dt_bias"]], tensors[p + nm["a_log"]], tensors[p + nm["skip"]]
+        self.norm_weight = tensors[p + nm["norm"]]
+        if self.out_scale != 1.0:
+            self.norm_weight = (self.norm_weight * self.out_scale).contiguous()
+
+    def forward(self, xb: torch.Tensor, residual: torch.Tensor, ctx, cache, write_cache: bool = True,
+                accumulate: bool = True) -> None:
+        n, dev, dt = xb.shape[0], xb.device, xb.dtype
+        I, C, H = self.inner, self.channels, self.H
+        proj = torch.empty((n, self.w_in.shape[0]), dtype=torch.float32, device=dev)
+        ops.gemm(xb, self.w_in, proj)
+        xbc = torch.empty((n, C), dtype=dt, device=dev)
+        self.conv.forward(proj[:, I:I + C], ctx, cache[1], xbc)
+        y = torch.empty((n, I), dtype=torch.float32, device=dev)
+        ops.state_space_scan(xbc, proj[:, I + C:I + C + H], self.dt_bias, self.a_log, self.skip, self._segments(ctx), cache[0].state,
+                             y, H, self.G, self.N, self.dv)
+        og = torch.empty((n, I), dtype=dt, device=dev)
+        ops.gated_part_norm(y, proj[:, :I], self.norm_weight, self.norm_eps, og, self.norm_groups)
+        ops.gemm(og, self.w_o, residual, accumulate=accumulate)
 
 
 class MLSTM(_SegmentScan):
@@ -393,3 +476,4 @@ register_part("mixer", "gated_delta_rule", GatedDeltaRule)
 register_part("mixer", "mlstm", MLSTM)
 register_part("mixer", "mingru", MinGRU)
 register_part("mixer", "retention", Retention)
+register_part("mixer", "state_space", StateSpace)
