@@ -823,12 +823,19 @@ def retention_scan(q, k, v, cos, sin, rotary_dim: int, positions, decay, segment
                                  _stream()), "retention_scan", launches=2)
 
 
+def state_space_chunks_take(state_dim: int, value_dim: int) -> bool:
+    """Whether the chunked form of `state_space_scan` takes a mixer of these sizes."""
+    return state_dim % 8 == 0 and state_dim <= 256 and value_dim % 8 == 0
+
+
 def state_space_scan(xbc, dt_logit, dt_bias, a_log, skip, segments, state, out, n_heads: int, n_groups: int, state_dim: int,
-                     value_dim: int) -> None:
+                     value_dim: int, long_segments=None) -> None:
     """The state-space recurrence over the rows of every segment, per head, S = state[slot, head] float32 (stored [dv, N]):
         dt = softplus(dt_logit + dt_bias);  S <- exp(-exp(a_log) dt) S + dt B x^T;  out = S^T C + skip x
     xbc [n, H*dv + 2*G*N] (a column slice, float32 or bfloat16) = [x | B | C]; head h reads group h // (H/G) of B and C;
-    dt_logit a float32 column slice [n, H]; dt_bias, a_log, skip float32 [H]; out float32 [n, H*dv]."""
+    dt_logit a float32 column slice [n, H]; dt_bias, a_log, skip float32 [H]; out float32 [n, H*dv].  `long_segments` int32
+    [n_long, 3] (bfloat16 xbc, sizes that `state_space_chunks_take`): these requests are walked in chunks of tokens as
+    matrix products on the tensor cores, those of `segments` token by token; a request stands in one of the two."""
     H, G, N, dv = n_heads, n_groups, state_dim, value_dim
     ldx = _cols(xbc, "xbc", H * dv + 2 * G * N, any_type=True)
     ldt = _cols(dt_logit, "dt_logit", H)
@@ -844,9 +851,17 @@ def state_space_scan(xbc, dt_logit, dt_bias, a_log, skip, segments, state, out, 
             or segments.shape[1] != 3:
         raise KernelError("state_space_scan: shapes do not fit")
     lib = build.load("state_space")
-    _check(lib.hk_state_space_walk(_ptr(xbc), _dt(xbc), ctypes.c_longlong(ldx), _ptr(dt_logit), ctypes.c_longlong(ldt), _ptr(dt_bias),
-                                   _ptr(a_log), _ptr(skip), _ptr(segments), int(segments.shape[0]), n, _ptr(state), _ptr(out), H, G, N,
-                                   dv, _stream()), "state_space_scan")
+    if long_segments is not None and long_segments.shape[0]:
+        _need(long_segments, "long_segments", torch.int32, 2)
+        if xbc.dtype != torch.bfloat16 or long_segments.shape[1] != 3:
+            raise KernelError("state_space_scan: long segments [n_long, 3] need bfloat16 rows")
+        _check(lib.hk_state_space_chunks(_ptr(xbc), ctypes.c_longlong(ldx), _ptr(dt_logit), ctypes.c_longlong(ldt), _ptr(dt_bias),
+                                         _ptr(a_log), _ptr(skip), _ptr(long_segments), int(long_segments.shape[0]), n, _ptr(state),
+                                         _ptr(out), H, G, N, dv, _stream()), "state_space_scan (chunks)")
+    if segments.shape[0]:
+        _check(lib.hk_state_space_walk(_ptr(xbc), _dt(xbc), ctypes.c_longlong(ldx), _ptr(dt_logit), ctypes.c_longlong(ldt), _ptr(dt_bias),
+                                       _ptr(a_log), _ptr(skip), _ptr(segments), int(segments.shape[0]), n, _ptr(state), _ptr(out), H, G,
+                                       N, dv, _stream()), "state_space_scan")
 
 
 def gated_part_norm(y, z, weight, eps: float, out, parts: int) -> None:

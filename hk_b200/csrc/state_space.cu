@@ -263,6 +263,380 @@ HK_API int hk_state_space_walk(const void* xbc, int dtype, long long ldx, const 
   return HK_ERR_UNSUPPORTED;
 }
 
+// ------------------------------------------------------------------ the walk, a chunk of tokens at a time (bf16 inputs)
+// The same recurrence for prompt portions as matrix products over chunks of 64 tokens, on mma.sync.  With the chunk's
+// cumulative log decays c_t (c_0 the first token's own) and its start state S_0, in exact arithmetic
+//     y_t = e^(c_t) S_0^T C_t + sum_(s <= t) e^(c_t - c_s) dt_s (C_t . B_s) x_s + D x_t
+//     S   = e^(c_last) S_0 + sum_s B_s (e^(c_last - c_s) dt_s x_s)^T
+// x, B and C are bf16 as they come and enter the products as they are; every float32 factor (the state, the weighted x, the
+// decayed scores) is cut into three bf16 numbers whose sum is the float32 number to its last bit or two, one product each,
+// with float32 sums.  The state stays in float32 registers from a portion's first chunk to its last.
+//
+// A block of eight warps owns DVB value columns of one head for one segment and walks its chunks in order, the next chunk's
+// rows on their way through cp.async meanwhile.  Warp w takes 16 of the 64 tokens (w & 3) and half of the columns (w >> 2)
+// of the outputs, and its share of the state's tiles (16 entries x 8 columns).
+namespace {
+
+constexpr int CQ = 64;      // tokens of a chunk
+
+__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, bool valid) {
+  const int bytes = valid ? 16 : 0;   // 0 source bytes: the 16 destination bytes are zero-filled
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void ldmatrix_x4(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldmatrix_x2_trans(uint32_t* r, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// two float32 numbers as three pairs of bf16 whose sums they are
+__device__ __forceinline__ void split3(float a, float b, uint32_t* out) {
+#pragma unroll
+  for (int p = 0; p < 3; ++p) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+    out[p] = *reinterpret_cast<const uint32_t*>(&v);
+    a -= __uint_as_float(out[p] << 16);
+    b -= __uint_as_float(out[p] & 0xffff0000u);
+  }
+}
+
+template <int NT, int DVB>
+struct ChunkShape {
+  static constexpr int LDN = NT + 8, LDX = DVB + 8;              // padded rows: an odd number of 16-byte pieces
+  static constexpr int RT = NT / 16;                             // state tiles of 16 entries
+  static constexpr int MT = RT > 8 ? RT / 8 : 1;                 // of which a warp holds MT ...
+  static constexpr int CP = RT < 8 ? 8 / RT : 1;                 // ... in 1 / CP of the columns,
+  static constexpr int NC = DVB / 8 / CP;                        // NC tiles of 8
+  static constexpr int NY = DVB / 16;                            // a warp's column tiles of the outputs
+  static constexpr size_t BC = (size_t)2 * 2 * CQ * LDN, X = (size_t)2 * CQ * LDX, XW = (size_t)3 * CQ * LDX, SS = (size_t)3 * NT * LDX;
+  static constexpr size_t SMEM = (BC + X + XW + SS) * sizeof(bf16) + 2 * CQ * sizeof(float2);
+};
+
+}  // namespace
+
+template <int NT, int DVB>
+__global__ void __launch_bounds__(256, 1)
+state_space_chunks_kernel(const bf16* __restrict__ xbc, long long ldx, const float* __restrict__ dt, long long ldt,
+                          const float* __restrict__ dt_bias, const float* __restrict__ a_log, const float* __restrict__ skip,
+                          const int* __restrict__ segs, float* __restrict__ state, float* __restrict__ y, int H, int G, int N, int dv) {
+  using K = ChunkShape<NT, DVB>;
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  bf16* bs = reinterpret_cast<bf16*>(smem_raw);       // [2][CQ][LDN]
+  bf16* cs = bs + 2 * CQ * K::LDN;                    // [2][CQ][LDN]
+  bf16* xs = cs + 2 * CQ * K::LDN;                    // [2][CQ][LDX]
+  bf16* xw = xs + K::X;                               // [3][CQ][LDX] the weighted x in three pieces
+  bf16* ss = xw + K::XW;                              // [3][NT][LDX] the chunk's start state in three pieces
+  float2* scal = reinterpret_cast<float2*>(ss + K::SS);     // [2][CQ] (cumulative log2 decay, step size)
+
+  const int seg = blockIdx.x / H, h = blockIdx.x % H;
+  const int slot = segs[seg * 3], row0 = segs[seg * 3 + 1], count = segs[seg * 3 + 2];
+  const int col0 = blockIdx.y * DVB, ncols = min(DVB, dv - col0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int qr = lane >> 2, qt = lane & 3, mi = lane >> 3, r8 = lane & 7;
+  const float bias = dt_bias[h], rate2 = expf(a_log[h]) * 1.4426950408889634f, dskip = skip[h];
+
+  // this warp's state tiles: rows (entries) st_row + 128 m + .., columns st_col + 8 c + ..
+  const int st_row = (warp % (K::RT < 8 ? K::RT : 8)) * 16, st_col = (K::RT < 8 ? warp / K::RT : 0) * K::NC * 8;
+  float* sp = state + (((size_t)slot * H + h) * dv + col0) * N;
+  float S[K::MT][K::NC][4];
+#pragma unroll
+  for (int m = 0; m < K::MT; ++m)
+#pragma unroll
+    for (int c = 0; c < K::NC; ++c)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = st_row + 128 * m + qr + 8 * (e >> 1), d = st_col + 8 * c + 2 * qt + (e & 1);
+        S[m][c][e] = n < N && d < ncols ? sp[(size_t)d * N + n] : 0.f;
+      }
+  auto publish = [&]() {                              // the state in three pieces, for everyone's read-out
+#pragma unroll
+    for (int m = 0; m < K::MT; ++m)
+#pragma unroll
+      for (int c = 0; c < K::NC; ++c)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          uint32_t piece[3];
+          split3(S[m][c][2 * i], S[m][c][2 * i + 1], piece);
+          bf16* d = ss + (size_t)(st_row + 128 * m + qr + 8 * i) * K::LDX + st_col + 8 * c + 2 * qt;
+#pragma unroll
+          for (int p = 0; p < 3; ++p) *reinterpret_cast<uint32_t*>(d + (size_t)p * NT * K::LDX) = piece[p];
+        }
+  };
+
+  const bf16* xg = xbc + (size_t)row0 * ldx + (size_t)h * dv + col0;
+  const bf16* bg = xbc + (size_t)row0 * ldx + (size_t)H * dv + (size_t)(h / (H / G)) * N;
+  const bf16* cg = bg + (size_t)G * N;
+  auto fetch = [&](int c) {                           // chunk c -> stage c & 1, rows and columns that do not exist as zeros
+    const int t0 = c * CQ, tc = min(CQ, count - t0);
+    bf16* db = bs + (size_t)(c & 1) * CQ * K::LDN;
+    bf16* dc = cs + (size_t)(c & 1) * CQ * K::LDN;
+    bf16* dx = xs + (size_t)(c & 1) * CQ * K::LDX;
+#pragma unroll
+    for (int i = 0; i < CQ * (NT / 8) / 256; ++i) {
+      const int e = tid + 256 * i, t = e / (NT / 8), p = (e % (NT / 8)) * 8;
+      const bool ok = t < tc && p < N;
+      const size_t src = ok ? (size_t)(t0 + t) * ldx + p : 0;
+      cp_async16_or_zero(db + t * K::LDN + p, bg + src, ok);
+      cp_async16_or_zero(dc + t * K::LDN + p, cg + src, ok);
+    }
+#pragma unroll
+    for (int i = 0; i < CQ * (DVB / 8) / 256; ++i) {
+      const int e = tid + 256 * i, t = e / (DVB / 8), p = (e % (DVB / 8)) * 8;
+      const bool ok = t < tc && p < ncols;
+      cp_async16_or_zero(dx + t * K::LDX + p, xg + (ok ? (size_t)(t0 + t) * ldx + p : 0), ok);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // warp 0 makes a chunk's scalars: lane l the tokens 2 l and 2 l + 1, their logits asked for a chunk ahead
+  float raw[2];
+  auto ask = [&](int c) {
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int t = c * CQ + 2 * lane + u;
+      raw[u] = t < count ? dt[(size_t)(row0 + t) * ldt + h] : 0.f;
+    }
+  };
+  auto scalars = [&](int c) {
+    float step[2], la[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      step[u] = c * CQ + 2 * lane + u < count ? softplus_f(raw[u] + bias) : 0.f;
+      la[u] = -rate2 * step[u];
+    }
+    const float own = la[0] + la[1];
+    float run = own;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += v;
+    }
+    float before = __shfl_up_sync(0xffffffffu, run, 1);
+    if (lane == 0) before = 0.f;
+    scal[(c & 1) * CQ + 2 * lane] = make_float2(before + la[0], step[0]);
+    scal[(c & 1) * CQ + 2 * lane + 1] = make_float2(run, step[1]);
+  };
+
+  const int nchunks = (count + CQ - 1) / CQ;
+  fetch(0);
+  if (warp == 0) {
+    ask(0);
+    scalars(0);
+  }
+  publish();
+  const int rg = warp & 3, yc = (warp >> 2) * (DVB / 2);       // this warp's tokens (16 rg ..) and output columns
+  const size_t ystep = (size_t)H * dv;
+  float* yp = y + (size_t)row0 * ystep + (size_t)h * dv + col0 + yc;
+  for (int c = 0; c < nchunks; ++c) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                  // the chunk's rows, scalars and start state are there
+    if (c + 1 < nchunks) {
+      fetch(c + 1);
+      if (warp == 0) ask(c + 1);
+    }
+    const bf16* bt = bs + (size_t)(c & 1) * CQ * K::LDN;
+    const bf16* ct = cs + (size_t)(c & 1) * CQ * K::LDN;
+    const bf16* xt = xs + (size_t)(c & 1) * CQ * K::LDX;
+    const float2* sc = scal + (c & 1) * CQ;
+    const float last = sc[CQ - 1].x;
+#pragma unroll
+    for (int i = 0; i < CQ * (DVB / 2) / 256; ++i) {
+      const int e = tid + 256 * i, t = e / (DVB / 2), d = (e % (DVB / 2)) * 2;
+      const uint32_t v = *reinterpret_cast<const uint32_t*>(xt + t * K::LDX + d);
+      const float w = exp2f(last - sc[t].x) * sc[t].y;
+      uint32_t piece[3];
+      split3(w * __uint_as_float(v << 16), w * __uint_as_float(v & 0xffff0000u), piece);
+#pragma unroll
+      for (int p = 0; p < 3; ++p) *reinterpret_cast<uint32_t*>(xw + (size_t)p * CQ * K::LDX + t * K::LDX + d) = piece[p];
+    }
+    __syncthreads();                                  // the weighted x is there
+
+    // ---- outputs: C S_0 over the entries, and the scores C B^T of this warp's tokens with the ones up to them
+    float acc[K::NY][4], g[4][2][4];
+#pragma unroll
+    for (int n = 0; n < K::NY; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) g[j][i][e] = 0.f;
+    const bf16* ca = ct + (rg * 16 + r8 + (mi & 1) * 8) * K::LDN + (mi >> 1) * 8;
+    const bf16* bb = bt + ((mi >> 1) * 8 + r8) * K::LDN + (mi & 1) * 8;
+    const bf16* sb = ss + (size_t)((mi & 1) * 8 + r8) * K::LDX + yc + (mi >> 1) * 8;
+#pragma unroll
+    for (int k = 0; k < NT / 16; ++k) {
+      uint32_t a[4];
+      ldmatrix_x4(a, ca + k * 16);
+#pragma unroll
+      for (int p = 0; p < 3; ++p)
+#pragma unroll
+        for (int np = 0; np < K::NY / 2; ++np) {
+          uint32_t b[4];
+          ldmatrix_x4_trans(b, sb + ((size_t)p * NT + k * 16) * K::LDX + np * 16);
+          mma_bf16(acc[2 * np], a, b[0], b[1]);
+          mma_bf16(acc[2 * np + 1], a, b[2], b[3]);
+        }
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (j <= rg) {
+          uint32_t b[4];
+          ldmatrix_x4(b, bb + j * 16 * K::LDN + k * 16);
+          mma_bf16(g[j][0], a, b[0], b[1]);
+          mma_bf16(g[j][1], a, b[2], b[3]);
+        }
+    }
+    const int t0 = rg * 16 + qr;
+    const float cum0 = sc[t0].x, cum1 = sc[t0 + 8].x;
+    {
+      const float f0 = exp2f(cum0), f1 = exp2f(cum1);
+#pragma unroll
+      for (int n = 0; n < K::NY; ++n) {
+        acc[n][0] *= f0;
+        acc[n][1] *= f0;
+        acc[n][2] *= f1;
+        acc[n][3] *= f1;
+      }
+    }
+    const bf16* xb = xt + ((mi & 1) * 8 + r8) * K::LDX + yc + (mi >> 1) * 8;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (j <= rg) {
+        uint32_t piece[4][3];                         // the decayed scores of 16 x 16 as an A fragment, in three pieces
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int s = j * 16 + i * 8 + 2 * qt;
+          const float2 s0 = sc[s], s1 = sc[s + 1];
+          const float m0 = s <= t0 ? g[j][i][0] * (exp2f(cum0 - s0.x) * s0.y) : 0.f;
+          const float m1 = s + 1 <= t0 ? g[j][i][1] * (exp2f(cum0 - s1.x) * s1.y) : 0.f;
+          const float m2 = s <= t0 + 8 ? g[j][i][2] * (exp2f(cum1 - s0.x) * s0.y) : 0.f;
+          const float m3 = s + 1 <= t0 + 8 ? g[j][i][3] * (exp2f(cum1 - s1.x) * s1.y) : 0.f;
+          split3(m0, m1, piece[2 * i]);
+          split3(m2, m3, piece[2 * i + 1]);
+        }
+#pragma unroll
+        for (int np = 0; np < K::NY / 2; ++np) {
+          uint32_t b[4];
+          ldmatrix_x4_trans(b, xb + j * 16 * K::LDX + np * 16);
+#pragma unroll
+          for (int p = 0; p < 3; ++p) {
+            const uint32_t a[4] = {piece[0][p], piece[1][p], piece[2][p], piece[3][p]};
+            mma_bf16(acc[2 * np], a, b[0], b[1]);
+            mma_bf16(acc[2 * np + 1], a, b[2], b[3]);
+          }
+        }
+      }
+    const int left = count - c * CQ;                  // tokens from the chunk's first on
+#pragma unroll
+    for (int n = 0; n < K::NY; ++n)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = t0 + 8 * i, d = n * 8 + 2 * qt;
+        if (t < left && yc + d < ncols) {
+          const uint32_t v = *reinterpret_cast<const uint32_t*>(xt + t * K::LDX + yc + d);
+          *reinterpret_cast<float2*>(yp + (size_t)(c * CQ + t) * ystep + d) =
+              make_float2(fmaf(dskip, __uint_as_float(v << 16), acc[n][2 * i]), fmaf(dskip, __uint_as_float(v & 0xffff0000u), acc[n][2 * i + 1]));
+        }
+      }
+
+    // ---- the state after the chunk
+    const float keep = exp2f(last);
+#pragma unroll
+    for (int m = 0; m < K::MT; ++m)
+#pragma unroll
+      for (int n = 0; n < K::NC; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[m][n][e] *= keep;
+    const bf16* ba = bt + ((mi >> 1) * 8 + r8) * K::LDN + st_row + (mi & 1) * 8;
+    const bf16* wb = xw + ((mi & 1) * 8 + r8) * K::LDX + st_col + (mi >> 1) * 8;
+#pragma unroll
+    for (int k = 0; k < CQ / 16; ++k) {
+      uint32_t a[K::MT][4];
+#pragma unroll
+      for (int m = 0; m < K::MT; ++m) ldmatrix_x4_trans(a[m], ba + k * 16 * K::LDN + 128 * m);
+#pragma unroll
+      for (int p = 0; p < 3; ++p) {
+        const bf16* w = wb + ((size_t)p * CQ + k * 16) * K::LDX;
+        if (K::NC == 1) {
+          uint32_t b[2];
+          ldmatrix_x2_trans(b, xw + ((size_t)p * CQ + k * 16 + (lane & 15)) * K::LDX + st_col);
+#pragma unroll
+          for (int m = 0; m < K::MT; ++m) mma_bf16(S[m][0], a[m], b[0], b[1]);
+        } else {
+#pragma unroll
+          for (int np = 0; np < K::NC / 2; ++np) {
+            uint32_t b[4];
+            ldmatrix_x4_trans(b, w + np * 16);
+#pragma unroll
+            for (int m = 0; m < K::MT; ++m) {
+              mma_bf16(S[m][2 * np], a[m], b[0], b[1]);
+              mma_bf16(S[m][2 * np + 1], a[m], b[2], b[3]);
+            }
+          }
+        }
+      }
+    }
+    if (c + 1 < nchunks) {
+      if (warp == 0) scalars(c + 1);
+      __syncthreads();                                // the start state is read: the next one may be published
+      publish();
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < K::MT; ++m)
+#pragma unroll
+    for (int c = 0; c < K::NC; ++c)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = st_row + 128 * m + qr + 8 * (e >> 1), d = st_col + 8 * c + 2 * qt + (e & 1);
+        if (n < N && d < ncols) sp[(size_t)d * N + n] = S[m][c][e];
+      }
+}
+
+template <int NT, int DVB>
+static int chunks_launch(const bf16* xbc, long long ldx, const float* dt, long long ldt, const float* dt_bias, const float* a_log,
+                         const float* skip, const int* segs, int n_seg, float* state, float* y, int H, int G, int N, int dv,
+                         cudaStream_t s) {
+  static HkSmemCache cache;
+  constexpr size_t smem = ChunkShape<NT, DVB>::SMEM;
+  if (int e = hk_allow_smem(state_space_chunks_kernel<NT, DVB>, smem, cache)) return e;
+  dim3 grid((unsigned)(n_seg * H), (unsigned)((dv + DVB - 1) / DVB));
+  return hk_launch(state_space_chunks_kernel<NT, DVB>, grid, dim3(256), smem, s, xbc, ldx, dt, ldt, dt_bias, a_log, skip, segs, state, y, H,
+                   G, N, dv);
+}
+
+// As hk_state_space_walk for bf16 rows, meant for segments of some length.  Refuses what the 16-byte copies cannot take (N,
+// dv or ldx no multiple of 8, an unaligned xbc) and states of more than 256 numbers a column.
+HK_API int hk_state_space_chunks(const void* xbc, long long ldx, const float* dt, long long ldt, const float* dt_bias,
+                                 const float* a_log, const float* skip, const int* segs, int n_seg, int n_rows, float* state, float* y,
+                                 int H, int G, int N, int dv, void* stream) {
+  if (n_seg <= 0 || n_rows <= 0) return 0;
+  if (H < 1 || G < 1 || H % G || N < 1 || N > 256 || (N & 7) || dv < 1 || (dv & 7) || (ldx & 7) || ((uintptr_t)xbc & 15)) return HK_ERR_UNSUPPORTED;
+  if ((uintptr_t)y & 7) return HK_ERR_UNSUPPORTED;
+  cudaStream_t s = (cudaStream_t)stream;
+#define CHUNKS(NT, DVB) chunks_launch<NT, DVB>((const bf16*)xbc, ldx, dt, ldt, dt_bias, a_log, skip, segs, n_seg, state, y, H, G, N, dv, s)
+  // 64 columns a block share the scores; 32 where that leaves SMs without a block
+  const bool wide = dv > 32 && (long long)n_seg * H * ((dv + 63) / 64) * 4 >= 3 * 148;
+  if (N <= 32) return wide ? CHUNKS(32, 64) : CHUNKS(32, 32);
+  if (N <= 64) return wide ? CHUNKS(64, 64) : CHUNKS(64, 32);
+  if (N <= 128) return wide ? CHUNKS(128, 64) : CHUNKS(128, 32);
+  return CHUNKS(256, 32);
+#undef CHUNKS
+}
+
 // ------------------------------------------------------------------ the gate, then a norm over equal parts of the row
 // u = y silu(z); each of `parts` equal parts of a row over its own root mean square (eps inside the root), times the
 // weight, narrowed to T.  A block per (token, part); the part's u stays in shared memory between the two passes.

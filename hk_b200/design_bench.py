@@ -365,7 +365,8 @@ def padodra_kernel_points(width: int, n: int, context: int, peaks: dict) -> dict
     cn = torch.ones(r, device=dev)
     cos = torch.ones(per + 1, dr // 2, device=dev)
     sin = torch.zeros(per + 1, dr // 2, device=dev)
-    us = _time_kernel(lambda: ops.latent_prep(proj, q_plain, ql, cn, 1e-6, cos, sin, dr, "half", positions, slot_of, table, rows_l,
+    at = H * (dn + dr)
+    us = _time_kernel(lambda: ops.latent_prep(proj[:, :at], proj[:, at:at + dk], q_plain, ql, cn, 1e-6, cos, sin, dr, "half", positions, slot_of, table, rows_l,
                                               H, dn, dr, r, pt))
     note("latent_prep", us, n * (H * (dn + dr) + dk) * 6, 0, 0, like="qk_norm_rope_kv_write (Qwen3)")
     qkv = torch.randn(n, (H + 2 * G) * hd, device=dev)
@@ -753,16 +754,241 @@ def zazulix_kernel_points(width: int, n: int, decode: bool, peaks: dict) -> dict
     return out
 
 
+def gezavik_shape(width: int, groups: int = 2, vocab: int = 32000, window: int = 1024) -> dict:
+    """Layer sizes that resemble a real model's: state-space layers of twice the width with heads of 64, states of 128,
+    eight groups and four taps; a latent attention with per head 128 plain and 64 rotated query dims, values of 128, a cached
+    latent of 512, queries through a latent of three eighths of the width and a window; a dense feed-forward of four times
+    the width and eight experts of half the width beside two identities, of which two are used, and a shared expert."""
+    heads, inner = width // 128, 2 * width
+    ssm = {"type": "mamba2", "mixer": {"heads": inner // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}}
+    lat = {"type": "latent_attention", "mixer": {"dim": 128, "heads": heads, "kv_rank": 512, "q_rank": 3 * width // 8, "rot_dim": 64,
+                                                 "vdim": 128, "mask": {"size": window}, "rot": {"base": 100000.0, "dims": 64},
+                                                 "scale": 1.0 / math.sqrt(192.0)}}
+    dense = {"kind": "dense", "ff": 4 * width}
+    moe = {"kind": "moe", "expert": {"ff": width // 2, "limit": 7.0}, "router": {"experts": 8, "identity": 2, "top": 2},
+           "shared": {"ff": width // 2, "limit": 7.0}}
+    layers = []
+    for g in range(groups):
+        layers += [dict(ssm, mlp=dense), dict(lat, mlp=moe), dict(ssm, mlp=moe), dict(ssm, mlp=moe)]
+    return {"architecture": "Gezavik", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": layers,
+            "initializer_range": 0.02}
+
+
+def gezavik_kernel_points(width: int, n: int, decode: bool, peaks: dict) -> dict:
+    """The design's kernels alone at a layer of this width, each beside the like kernel of the Zazulix (or Padodra)
+    decoder: one request of n prompt tokens, or (decode) n requests that each bring one token (the attention over the last
+    1,024 of 2,047 cached ones; these are timed as replays of a captured graph)."""
+    import numpy as np
+    import torch
+
+    from .csrc import attention_fast, gemm_fast, ops
+    dev = "cuda"
+    bw, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    out = {}
+
+    def note(name, us, nbytes, flops, peak_flops, like=None):
+        floor = max(nbytes / bw, flops / peak_flops if peak_flops else 0.0) * 1e6
+        out[name] = {"us": round(us, 1), "bytes": int(nbytes), "flops": int(flops), "roofline_us": round(floor, 2),
+                     "of_roofline": round(floor / us, 3), **({"like": like} if like else {})}
+
+    count, rows = (n, 1) if decode else (1, n)
+    _time_kernel = lambda fn: globals()["_time_kernel"](fn, replay=decode)      # decode steps replay a captured graph
+    sg = torch.tensor([[i, i * rows, rows] for i in range(count)], dtype=torch.int32, device=dev)
+    fp32 = FP32_TFLOPS * 1e12
+    bf = torch.bfloat16
+
+    # ---- the state-space mixer: convolution, recurrence, gated norm
+    H, dv, N, G, taps, parts = width // 32, 64, 128, 8, 4, 8
+    I, C = H * dv, H * dv + 2 * G * N
+    proj = torch.randn(n, -(-(I + C + H) // 8) * 8, device=dev) * 0.5
+    wconv = torch.randn(C, taps, device=dev) * 0.3
+    bconv = torch.randn(C, device=dev) * 0.1
+    tail = torch.zeros(count, taps - 1, C, device=dev)
+    xbc = torch.empty(n, C, dtype=bf, device=dev)
+    us = _time_kernel(lambda: ops.short_conv(proj[:, I:I + C], wconv, sg, tail, xbc, bias=bconv))
+    note("short_conv (x, B and C: bias, silu, bf16 out)", us, n * C * 6 + count * (taps - 1) * C * 8, 2.0 * n * C * taps, fp32,
+         like="short_conv (Zazulix: no bias, no activation, float32 out)")
+    xf = torch.empty(n, C, device=dev)
+    us = _time_kernel(lambda: ops.short_conv(proj[:, I:I + C], wconv, sg, tail, xf, act="none"))
+    note("short_conv (Zazulix: no bias, no activation, float32 out)", us, n * C * 8 + count * (taps - 1) * C * 8, 2.0 * n * C * taps, fp32)
+    del xf
+    dtb = torch.full((H,), -4.0, device=dev)
+    alog = torch.zeros(H, device=dev)
+    skip = torch.ones(H, device=dev)
+    state = torch.zeros(count, H, dv, N, device=dev)
+    y = torch.empty(n, I, device=dev)
+    none = sg[:0]
+    short, chunked = (sg, none) if decode else (none, sg)
+    us = _time_kernel(lambda: ops.state_space_scan(xbc, proj[:, I + C:I + C + H], dtb, alog, skip, short, state, y, H, G, N, dv,
+                                                   long_segments=chunked))
+    # decode walks token by token (fp32 FMA peak); a prompt's chunks run on the tensor cores, where the bytes are the floor
+    note("state_space_scan", us, n * (C * 2 + H * 4 + I * 4) + 8 * count * H * dv * N, 4.0 * n * H * dv * N, fp32 if decode else tc,
+         like="retention_scan (Zazulix)")
+    if not decode:
+        us = _time_kernel(lambda: ops.state_space_scan(xbc, proj[:, I + C:I + C + H], dtb, alog, skip, sg, state, y, H, G, N, dv))
+        note("state_space_scan, token by token", us, n * (C * 2 + H * 4 + I * 4) + 8 * count * H * dv * N, 4.0 * n * H * dv * N, fp32,
+             like="retention_scan (Zazulix)")
+    # the like scan at as many state entries: heads of 64 x 64, twice as many
+    Hr, dr_ = 2 * H, 64
+    KK = Hr * dr_
+    projr = torch.randn(n, 3 * KK, device=dev) * 0.5
+    state_r = torch.zeros(count, Hr, dr_, dr_, device=dev)
+    o = torch.empty(n, KK, device=dev)
+    decay = torch.full((Hr,), 0.99, device=dev)
+    zero_pos = torch.zeros(n, dtype=torch.int32, device=dev)
+    us = _time_kernel(lambda: ops.retention_scan(projr[:, :KK], projr[:, KK:2 * KK], projr[:, 2 * KK:], None, None, 0, zero_pos, decay, sg,
+                                                 state_r, o, Hr, dr_, dr_, dr_ ** -0.5))
+    note("retention_scan (Zazulix)", us, 4 * (4 * n * KK + 2 * count * Hr * dr_ * dr_), 4.0 * n * Hr * dr_ * dr_, fp32)
+    del projr, state_r, state
+    wn = torch.ones(I, device=dev)
+    og = torch.empty(n, I, dtype=bf, device=dev)
+    us = _time_kernel(lambda: ops.gated_part_norm(y, proj[:, :I], wn, 1e-6, og, parts))
+    note("gated_part_norm", us, n * I * (4 + 4 + 2), 0, 0, like="head_out_gate (Zazulix: no weight, silu)")
+    us = _time_kernel(lambda: ops.head_out_gate(y, proj[:, :I], None, 1e-6, og, H, dv, act="silu"))
+    note("head_out_gate (Zazulix: no weight, silu)", us, n * I * (4 + 4 + 2), 0, 0)
+
+    # ---- latent attention: the query latent's norm, what a token brings, the attention, the per-head products
+    Ha, r, dr, dn, vd, pt, context, window, qr = width // 128, 512, 64, 128, 128, 64, 2047, 1024, 3 * width // 8
+    dk = r + dr
+    sm = torch.cuda.get_device_properties(0).multi_processor_count
+    per = (context + 1) if decode else n
+    ppr = -(-per // pt)
+    table = torch.arange(count * ppr, dtype=torch.int32, device=dev).view(count, ppr).contiguous()
+    slots = list(range(count))
+    q_starts, q_lens = (list(range(n)), [1] * n) if decode else ([0], [n])
+    starts = [context] * n if decode else [0]
+    positions = torch.tensor([context] * n if decode else list(range(n)), dtype=torch.int32, device=dev)
+    slot_of = torch.tensor(list(range(n)) if decode else [0] * n, dtype=torch.int32, device=dev)
+    up = lambda a: torch.from_numpy(np.ascontiguousarray(a)).to(dev)
+    seen = [min(p + 1, window) for p in ([context] * n if decode else range(n))]
+    rows_l = (torch.randn(count * ppr, 1, pt, dk, device=dev) * 0.3).bfloat16()
+    ql = (torch.randn(n, Ha * dk, device=dev) * 0.3).bfloat16()
+    lat = torch.empty(n, Ha * r, dtype=bf, device=dev)
+    plan = attention_fast.build_plan(slots, q_starts, q_lens, starts, n, window, Ha, 1, sm, up,
+                                     fixed_splits=attention_fast.decode_splits(n, 1, sm) if decode else 0,
+                                     max_context=context + 64 if decode else 0, prefill_rows=64)
+    us = _time_kernel(lambda: attention_fast.run_latent(ql, rows_l, table, lat, Ha, dk, r, pt, window, 192 ** -0.5, plan, single_tokens=decode))
+    note("latent attention (rows of 576, window)", us, (sum(seen) if decode else n) * dk * 2 + n * Ha * (dk + r) * 2,
+         2.0 * sum(seen) * Ha * (dk + r), tc, like="latent attention (Zazulix: rows of 512, window)")
+    rows_z = rows_l.view(-1)[:count * ppr * pt * r].view(count * ppr, 1, pt, r)
+    qz = ql.view(-1)[:n * Ha * r].view(n, Ha * r)
+    us = _time_kernel(lambda: attention_fast.run_latent(qz, rows_z, table, lat, Ha, r, r, pt, window, 128 ** -0.5, plan, single_tokens=decode))
+    note("latent attention (Zazulix: rows of 512, window)", us, (sum(seen) if decode else n) * r * 2 + n * Ha * 2 * r * 2,
+         2.0 * sum(seen) * Ha * 2 * r, tc)
+    lp = torch.randn(n, -(-(qr + dk + Ha) // 8) * 8, device=dev)
+    cq = torch.empty(n, qr, dtype=bf, device=dev)
+    wq = torch.ones(qr, device=dev)
+    us = _time_kernel(lambda: ops.rms_norm(lp[:, :qr], wq, 1e-6, cq))
+    note("rms_norm of the query latent (a column slice)", us, n * qr * 6, 0, 0, like="rms_norm (whole rows of the width)")
+    x = torch.randn(n, width, device=dev)
+    wx = torch.ones(width, device=dev)
+    xb = torch.empty(n, width, dtype=bf, device=dev)
+    us = _time_kernel(lambda: ops.rms_norm(x, wx, 1e-6, xb))
+    note("rms_norm (whole rows of the width)", us, n * width * 6, 0, 0)
+    qf = torch.randn(n, Ha * (dn + dr), device=dev)
+    q_plain = torch.empty(n, Ha * dn, dtype=bf, device=dev)
+    cn = torch.ones(r, device=dev)
+    cos = torch.ones(per + 1, dr // 2, device=dev)
+    sin = torch.zeros(per + 1, dr // 2, device=dev)
+    us = _time_kernel(lambda: ops.latent_prep(qf, lp[:, qr:qr + dk], q_plain, ql, cn, 1e-6, cos, sin, dr, "adjacent", positions, slot_of,
+                                              table, rows_l, Ha, dn, dr, r, pt))
+    note("latent_prep (queries and rows from two matrices)", us, n * (Ha * (dn + dr) + dk) * 6, 0, 0, like="latent_prep (Padodra: one matrix)")
+    both = torch.randn(n, Ha * (dn + dr) + dk, device=dev)
+    us = _time_kernel(lambda: ops.latent_prep(both[:, :Ha * (dn + dr)], both[:, Ha * (dn + dr):], q_plain, ql, cn, 1e-6, cos, sin, dr, "half",
+                                              positions, slot_of, table, rows_l, Ha, dn, dr, r, pt))
+    note("latent_prep (Padodra: one matrix)", us, n * (Ha * (dn + dr) + dk) * 6, 0, 0)
+    w_uv = (torch.randn(Ha, vd, r, device=dev) * 0.05).bfloat16()
+    ob = torch.empty(n, Ha * vd, dtype=bf, device=dev)
+    us = _time_kernel(lambda: ops.gemm_heads(lat.view(n, Ha, r), w_uv, ob.view(n, Ha, vd), Ha, gate=lp[:, qr + dk:qr + dk + Ha],
+                                             gate_scale=0.5, gate_per_head=True))
+    note("values out of the latent space, one gate a head", us, Ha * r * vd * 2 + n * Ha * (r * 2 + vd * 2), 2.0 * n * Ha * r * vd, tc,
+         like="values out of the latent space, element-wise gate (Zazulix)")
+    glat = torch.randn(n, Ha * vd, device=dev)
+    us = _time_kernel(lambda: ops.gemm_heads(lat.view(n, Ha, r), w_uv, ob.view(n, Ha, vd), Ha, gate=glat))
+    note("values out of the latent space, element-wise gate (Zazulix)", us, Ha * r * vd * 2 + n * Ha * (r * 2 + vd * 6), 2.0 * n * Ha * r * vd, tc)
+
+    # ---- the router over all outputs, the experts' products with the clamped activation, the combination
+    E, ident, top, Fe = 8, 2, 2, width // 2
+    xb.copy_(torch.randn(n, width, device=dev) * 0.5)
+    wr = torch.randn(E + ident, width, device=dev) * 0.05
+    corr = torch.randn(E + ident, device=dev) * 0.02
+    ids = torch.empty(n, top, dtype=torch.int32, device=dev)
+    wts = torch.empty(n, top, device=dev)
+    us = _time_kernel(lambda: ops.route_topk(xb, wr, ids, wts, "sigmoid", corr, 2, 1, 1.0, 1e-20))
+    note("route_topk (Zazulix: sigmoid scores, groups)", us, n * width * 2 + (E + ident) * width * 4, 2.0 * n * (E + ident) * width, fp32)
+    us = _time_kernel(lambda: ops.route_topk(xb, wr, ids, wts, "softmax_all", corr))
+    note("route_topk (softmax over all, correction, identities)", us, n * width * 2 + (E + ident) * width * 4, 2.0 * n * (E + ident) * width, fp32,
+         like="route_topk (Zazulix: sigmoid scores, groups)")
+    real = int((ids < E).sum())
+    pairs = n * top
+    wgu = (torch.randn(E, 2 * Fe, width, device=dev) * 0.02).bfloat16()
+    used = min(E, pairs)
+    nbytes, flops = used * 2 * Fe * width * 2 + real * (width + Fe) * 2, 2.0 * real * 2 * Fe * width
+    if pairs >= 1024:
+        pad = gemm_fast.GROUPED_ROWS
+        m_max = -(-(pairs + E * (pad - 1)) // pad) * pad
+        perm = torch.empty(m_max, dtype=torch.int32, device=dev)
+        inv = torch.empty(pairs, dtype=torch.int32, device=dev)
+        tiles = torch.empty(m_max // pad, dtype=torch.int32, device=dev)
+        ops.route_sort_padded(ids, E, pad, perm, inv, tiles)
+        xs = torch.empty(m_max, width, dtype=bf, device=dev)
+        ops.route_gather(xb, perm, top, xs)
+        h = torch.empty(m_max, Fe, dtype=bf, device=dev)
+        ys = torch.randn(m_max, width, device=dev)
+        grouped = lambda act: ops.grouped_gemm_tc(xs, wgu, h, tiles, gated=True, act=act, limit=7.0, slope=1.702)
+    else:
+        max_tiles = pairs // ops.route_tile_rows() + min(E, pairs)
+        offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
+        perm = torch.empty(pairs, dtype=torch.int32, device=dev)
+        inv = torch.empty(pairs, dtype=torch.int32, device=dev)
+        tiles = torch.empty(max_tiles, 2, dtype=torch.int32, device=dev)
+        ops.route_sort(ids, E, offsets, perm, inv, tiles)
+        h = torch.empty(pairs, Fe, dtype=bf, device=dev)
+        ys = torch.randn(pairs, width, device=dev)
+        grouped = lambda act: ops.grouped_gemm(xb, wgu, h, tiles, offsets, perm, top, gather=True, gated=True, act=act, limit=7.0, slope=1.702)
+    us = _time_kernel(lambda: grouped("swish_clamped"))
+    note("grouped gate/up product, clamped activation", us, nbytes, flops, tc, like="grouped gate/up product, silu (Zazulix)")
+    us = _time_kernel(lambda: grouped("silu"))
+    note("grouped gate/up product, silu (Zazulix)", us, nbytes, flops, tc)
+    res = torch.randn(n, width, device=dev)
+    shared = torch.randn(n, width, device=dev)
+    us = _time_kernel(lambda: ops.route_combine(ys, inv, wts, res, accumulate=True, shared=shared, x=xb, factor=0.5))
+    note("route_combine (identities, shared expert, factor)", us, n * width * 4 * 3 + real * width * 4 + (pairs - real) * width * 2, 0, 0,
+         like="route_combine (Zazulix)")
+    us = _time_kernel(lambda: ops.route_combine(ys, inv.clamp_min(0), wts, res, accumulate=True, shared=shared))
+    note("route_combine (Zazulix)", us, n * width * 4 * (top + 3), 0, 0)
+
+    # ---- the dense feed-forward's first product with the squared relu, beside the gated one of as many weights
+    F = 4 * width
+    w_up = (torch.randn(F, width, device=dev) * 0.02).bfloat16()
+    hb = torch.empty(n, F, dtype=bf, device=dev)
+    us = _time_kernel(lambda: ops.gemm_squared_relu(xb, w_up, hb, 0.5))
+    note("up product with the squared relu", us, F * width * 2 + n * (width + F) * 2, 2.0 * n * F * width, tc,
+         like="gate/up product, clamped (Zazulix)")
+    hz = torch.empty(n, F // 2, dtype=bf, device=dev)
+    us = _time_kernel(lambda: ops.gemm_swiglu(xb, w_up, hz, "swish_clamped", 7.0, 1.702))
+    note("gate/up product, clamped (Zazulix)", us, F * width * 2 + n * (width + F // 2) * 2, 2.0 * n * F * width, tc)
+    return out
+
+
+# design -> (its shape, the closest other design and its shape by width and layer runs)
+BESIDE = {"mifolorn": ("kedanex", lambda width, runs: kedanex_shape(width, runs // 4)),
+          "zazulix": ("kedanex", lambda width, runs: kedanex_shape(width, runs // 4)),
+          "gezavik": ("zazulix", lambda width, runs: zazulix_shape(width, runs // 4))}
+SHAPES = {"kedanex": kedanex_shape, "padodra": padodra_shape, "mifolorn": mifolorn_shape, "zazulix": zazulix_shape, "gezavik": gezavik_shape}
+
+
 def run(design: str, args, peaks: dict) -> dict:
-    if design not in ("kedanex", "padodra", "mifolorn", "zazulix"):
-        raise SystemExit(f"bench.py --design: unknown design '{design}' (known: kedanex, padodra, mifolorn, zazulix)")
+    if design not in SHAPES:
+        raise SystemExit(f"bench.py --design: unknown design '{design}' (known: {', '.join(SHAPES)})")
     widths = [int(w) for w in str(args.design_widths).split(",")]
     sizes = {}
     for width in widths:
         t0 = time.time()
-        ours = {"kedanex": kedanex_shape, "padodra": padodra_shape, "mifolorn": mifolorn_shape, "zazulix": zazulix_shape}[design](width)
+        ours = SHAPES[design](width)
         runs = len(ours["layers"]) * (ours["loop"]["times"] if "loop" in ours else 1)
-        beside, theirs = ("kedanex", kedanex_shape(width, runs // 4)) if design in ("mifolorn", "zazulix") else ("qwen3", qwen3_shape(width, runs))
+        beside, shape_of = BESIDE.get(design, ("qwen3", qwen3_shape))
+        theirs = shape_of(width, runs)
         entry = {design: model_points(ours, 2048, (8, 64), args.steps, max(args.warmup, 3), 5),
                  beside: model_points(theirs, 2048, (8, 64), args.steps, max(args.warmup, 3), 5),
                  "layer_runs": runs}
@@ -772,6 +998,9 @@ def run(design: str, args, peaks: dict) -> dict:
         elif design == "zazulix":
             entry["kernels_prefill_2048_rows"] = zazulix_kernel_points(width, 2048, False, peaks)
             entry["kernels_decode_64_rows"] = zazulix_kernel_points(width, 64, True, peaks)
+        elif design == "gezavik":
+            entry["kernels_prefill_2048_rows"] = gezavik_kernel_points(width, 2048, False, peaks)
+            entry["kernels_decode_64_rows"] = gezavik_kernel_points(width, 64, True, peaks)
         elif design == "kedanex":
             entry["kernels_prefill_2048_rows"] = kernel_points(width, 2048, peaks)
             entry["kernels_decode_64_rows"] = {k: v for k, v in kernel_points(width, 64, peaks).items() if "request" not in k or "decode" in k}
@@ -782,7 +1011,7 @@ def run(design: str, args, peaks: dict) -> dict:
         sizes[f"width{width}"] = entry
         print(f"[bench] design {design}, width {width}: {time.time() - t0:.0f} s", file=sys.stderr, flush=True)
     k = sizes[f"width{widths[-1]}"]
-    return {"metric": f"{design} prefill and decode tok/s beside {'Kedanex' if design in ('mifolorn', 'zazulix') else 'Qwen3'} at equal width and depth", "value": k[design]["decode_b8"]["tok_s"],
+    return {"metric": f"{design} prefill and decode tok/s beside {BESIDE.get(design, ('qwen3',))[0].capitalize()} at equal width and depth", "value": k[design]["decode_b8"]["tok_s"],
             "unit": "tokens/s (decode, batch 8, largest width)", "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3),
             "higher_is_better": True, "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random-init weights",
             "impl": "ours", "design": design, "sizes": sizes, "peaks": peaks}

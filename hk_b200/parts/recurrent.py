@@ -353,8 +353,12 @@ class ShortConvolution(_SegmentScan):
 
 class StateSpace(_SegmentScan):
     """`out_scale` is a factor on the mixer's result (carried by the norm's weight).  The input projection's one tensor is
-    the product's weight as it is, filled up to a multiple of 8 rows."""
+    the product's weight as it is, filled up to a multiple of 8 rows.  When serving in bfloat16, a request that brings
+    `CHUNKS_FROM` tokens or more to a step is walked in chunks of tokens on the tensor cores (`ops.state_space_scan`), the
+    others token by token; the two lists of requests are this part's host-built tables."""
     kernel_libraries = ("state_space",)
+    CHUNKS_FROM = 32
+    SPLIT_KEY = ("state_space_segments",)
 
     def __init__(self, hidden: int, n_heads: int, value_dim: int, state_dim: int, n_groups: int, taps: int, prefix: str,
                  norm_eps: float, norm_groups: int = 1, out_scale: float = 1.0, names: Optional[Dict[str, str]] = None):
@@ -368,6 +372,18 @@ class StateSpace(_SegmentScan):
         self.names.update(names or {})
         self.conv = ShortConvolution([(prefix + self.names["conv"], self.channels)], taps, act="silu", bias=True)
         self.w_in = self.w_o = self.dt_bias = self.a_log = self.skip = self.norm_weight = None
+        self._chunks = False            # set at bind: the chunked walk takes this mixer's sizes
+
+    def step_tables_key(self):
+        return self.SPLIT_KEY if self._chunks else SEGMENTS_KEY
+
+    def step_tables(self, ctx):
+        tables = segment_tables(ctx)
+        if not self._chunks:
+            return tables
+        seg = tables.arrays["segments"]
+        chunked = seg[:, 2] >= self.CHUNKS_FROM
+        return StepTables({"short": seg[~chunked], "long": seg[chunked]})
 
     @property
     def inner(self) -> int:
@@ -400,6 +416,7 @@ class StateSpace(_SegmentScan):
         self.norm_weight = tensors[p + nm["norm"]]
         if self.out_scale != 1.0:
             self.norm_weight = (self.norm_weight * self.out_scale).contiguous()
+        self._chunks = precision.compute == torch.bfloat16 and ops.state_space_chunks_take(self.N, self.dv)
 
     def forward(self, xb: torch.Tensor, residual: torch.Tensor, ctx, cache, write_cache: bool = True,
                 accumulate: bool = True) -> None:
@@ -410,8 +427,10 @@ class StateSpace(_SegmentScan):
         xbc = torch.empty((n, C), dtype=dt, device=dev)
         self.conv.forward(proj[:, I:I + C], ctx, cache[1], xbc)
         y = torch.empty((n, I), dtype=torch.float32, device=dev)
-        ops.state_space_scan(xbc, proj[:, I + C:I + C + H], self.dt_bias, self.a_log, self.skip, self._segments(ctx), cache[0].state,
-                             y, H, self.G, self.N, self.dv)
+        arrays = ctx.tables[self.step_tables_key()][0]
+        ops.state_space_scan(xbc, proj[:, I + C:I + C + H], self.dt_bias, self.a_log, self.skip,
+                             arrays["short" if self._chunks else "segments"], cache[0].state, y, H, self.G, self.N, self.dv,
+                             long_segments=arrays.get("long"))
         og = torch.empty((n, I), dtype=dt, device=dev)
         ops.gated_part_norm(y, proj[:, :I], self.norm_weight, self.norm_eps, og, self.norm_groups)
         ops.gemm(og, self.w_o, residual, accumulate=accumulate)
