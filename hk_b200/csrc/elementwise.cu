@@ -200,8 +200,9 @@ HK_API int hk_rms_norm(const float* x, const float* w, const int* rows, void* ou
                        int n_out, int d, long long ldx, float eps, void* stream) {
   if (n_out <= 0) return 0;
   cudaStream_t s = (cudaStream_t)stream;
-  if ((d & 3) == 0 && (ldx & 3) == 0 && d >= 1024 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0) {
+  if ((d & 3) == 0 && (ldx & 3) == 0 && d >= 256 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0) {
     const int chunks = d >> 2;
+    if (chunks <= 256) return rms_norm_vec<1>(x, w, rows, out, out_dtype, n_out, d, ldx, eps, s);
     if (chunks <= 2 * 256) return rms_norm_vec<2>(x, w, rows, out, out_dtype, n_out, d, ldx, eps, s);
     if (chunks <= 4 * 256) return rms_norm_vec<4>(x, w, rows, out, out_dtype, n_out, d, ldx, eps, s);
     if (chunks <= 8 * 256) return rms_norm_vec<8>(x, w, rows, out, out_dtype, n_out, d, ldx, eps, s);

@@ -835,7 +835,8 @@ def state_space_scan(xbc, dt_logit, dt_bias, a_log, skip, segments, state, out, 
     xbc [n, H*dv + 2*G*N] (a column slice, float32 or bfloat16) = [x | B | C]; head h reads group h // (H/G) of B and C;
     dt_logit a float32 column slice [n, H]; dt_bias, a_log, skip float32 [H]; out float32 [n, H*dv].  `long_segments` int32
     [n_long, 3] (bfloat16 xbc, sizes that `state_space_chunks_take`): these requests are walked in chunks of tokens as
-    matrix products on the tensor cores, those of `segments` token by token; a request stands in one of the two."""
+    matrix products on the tensor cores, those of `segments` token by token; a request stands in one of the two, and the
+    requests' rows are all of xbc's."""
     H, G, N, dv = n_heads, n_groups, state_dim, value_dim
     ldx = _cols(xbc, "xbc", H * dv + 2 * G * N, any_type=True)
     ldt = _cols(dt_logit, "dt_logit", H)
@@ -861,7 +862,7 @@ def state_space_scan(xbc, dt_logit, dt_bias, a_log, skip, segments, state, out, 
     if segments.shape[0]:
         _check(lib.hk_state_space_walk(_ptr(xbc), _dt(xbc), ctypes.c_longlong(ldx), _ptr(dt_logit), ctypes.c_longlong(ldt), _ptr(dt_bias),
                                        _ptr(a_log), _ptr(skip), _ptr(segments), int(segments.shape[0]), n, _ptr(state), _ptr(out), H, G,
-                                       N, dv, _stream()), "state_space_scan")
+                                       N, dv, 1 if segments.shape[0] == n else 0, _stream()), "state_space_scan")
 
 
 def gated_part_norm(y, z, weight, eps: float, out, parts: int) -> None:

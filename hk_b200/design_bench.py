@@ -879,12 +879,11 @@ def gezavik_kernel_points(width: int, n: int, decode: bool, peaks: dict) -> dict
     cq = torch.empty(n, qr, dtype=bf, device=dev)
     wq = torch.ones(qr, device=dev)
     us = _time_kernel(lambda: ops.rms_norm(lp[:, :qr], wq, 1e-6, cq))
-    note("rms_norm of the query latent (a column slice)", us, n * qr * 6, 0, 0, like="rms_norm (whole rows of the width)")
-    x = torch.randn(n, width, device=dev)
-    wx = torch.ones(width, device=dev)
+    note("rms_norm of the query latent (a column slice)", us, n * qr * 6, 0, 0, like="rms_norm (whole rows as wide)")
+    x = torch.randn(n, qr, device=dev)
+    us = _time_kernel(lambda: ops.rms_norm(x, wq, 1e-6, cq))
+    note("rms_norm (whole rows as wide)", us, n * qr * 6, 0, 0)
     xb = torch.empty(n, width, dtype=bf, device=dev)
-    us = _time_kernel(lambda: ops.rms_norm(x, wx, 1e-6, xb))
-    note("rms_norm (whole rows of the width)", us, n * width * 6, 0, 0)
     qf = torch.randn(n, Ha * (dn + dr), device=dev)
     q_plain = torch.empty(n, Ha * dn, dtype=bf, device=dev)
     cn = torch.ones(r, device=dev)
