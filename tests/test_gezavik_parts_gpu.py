@@ -156,6 +156,29 @@ def test_chunked_walk_is_the_token_walk_in_32_bit(H, G, N, dv, step_shift):
         assert torch.equal(state[0], start[0])     # the slot of no request
 
 
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("H,G,N,dv", [(4, 2, 128, 64), (3, 1, 32, 20), (2, 2, 64, 5), (2, 1, 200, 8), (1, 1, 300, 12), (1, 1, 516, 8), (100, 1, 16, 64)])
+def test_single_token_steps_equal_the_walk_bit_for_bit(dtype, H, G, N, dv):
+    """A step of single tokens runs a kernel of its own; beside one portion of two tokens the same requests go through the
+    ring.  Logits may not depend on which."""
+    from hk_b200.csrc import ops
+    reqs, inner = 5, H * dv
+    C = inner + 2 * G * N
+    xbc = (torch.randn(reqs + 2, C, device="cuda") * 0.7).to(dtype)
+    dt = torch.randn(reqs + 2, H, device="cuda")
+    dt_bias, a_log, skip = (torch.randn(H, device="cuda") * 0.5 for _ in range(3))
+    start = torch.randn(reqs + 1, H, dv, N, device="cuda")
+    segs = torch.tensor([[reqs - i, i, 1] for i in range(reqs)] + [[0, reqs, 2]], dtype=torch.int32, device="cuda")
+    alone, beside = start.clone(), start.clone()
+    y1, y2 = torch.full((reqs, inner), float("nan"), device="cuda"), torch.full((reqs + 2, inner), float("nan"), device="cuda")
+    ops.state_space_scan(xbc[:reqs], dt[:reqs], dt_bias, a_log, skip, segs[:reqs].contiguous(), alone, y1, H, G, N, dv)
+    ops.state_space_scan(xbc, dt, dt_bias, a_log, skip, segs, beside, y2, H, G, N, dv)
+    assert torch.equal(y1, y2[:reqs]) and torch.equal(alone[1:], beside[1:]) and torch.equal(alone[0], start[0])
+    for slot, r0, l in segs.tolist():
+        want, S = walk_in_double(xbc[r0:r0 + l], dt[r0:r0 + l], dt_bias, a_log, skip, start[slot], H, G, N, dv)
+        assert (y2[r0:r0 + l] - want).abs().max() <= 3e-6 * want.abs().max() and (beside[slot] - S).abs().max() <= 3e-6 * S.abs().max()
+
+
 # ------------------------------------------------------------------------------------ latent attention
 
 def latent_part(d, H, dn, dr, vd, qr, r, rot, window, scale, positions=512):
