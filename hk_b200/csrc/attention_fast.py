@@ -210,7 +210,7 @@ GATED = 2       # what `run` returns when the kernel it took also applied the ou
 
 def run(q, k_pages, v_pages, block_table, out, H, G, hd, page_tokens, window, scale, plan: FlashPlan,
         allow_tma: bool = True, sink: bool = False, sinks=None, softcap: float = 0.0, chunk: int = 0, gate=None,
-        gate_scale: float = 1.0):
+        gate_scale: float = 1.0, dist=None):
     """Runs the step on the flash kernels.  Returns False when they refuse it, True when `out` holds the attention, and
     GATED when it holds the attention times gate_scale * sigmoid(gate) (the tcgen05 prompt kernels apply a gate whose
     rows are 16-byte aligned in their epilogue; after any other kernel the caller applies it)."""
@@ -219,6 +219,7 @@ def run(q, k_pages, v_pages, block_table, out, H, G, hd, page_tokens, window, sc
         return False
     sk = 1 if sink else 0
     extra = (_ptr(sinks), ctypes.c_float(softcap), int(chunk))
+    bias = (_ptr(dist), int(dist.shape[1]) if dist is not None else 0)      # per query head and distance, in the base-2 domain
     fused_gate = gate is not None and gate.data_ptr() % 16 == 0 and gate.stride(0) % 4 == 0 and gate.stride(1) == 1
     gate_args = (_ptr(gate if fused_gate else None), ctypes.c_longlong(gate.stride(0) if fused_gate else 0), ctypes.c_float(gate_scale))
     done = GATED if fused_gate else True
@@ -237,7 +238,7 @@ def run(q, k_pages, v_pages, block_table, out, H, G, hd, page_tokens, window, sc
             _ptr(q), _ptr(k_pages), _ptr(v_pages), ctypes.c_longlong(k_pages.shape[0]), _ptr(block_table),
             int(block_table.shape[1]), _ptr(plan.items), plan.n_items, _ptr(out), H, G, hd, int(page_tokens), int(window),
             ctypes.c_float(scale * math.log2(math.e)), plan.max_keys // int(page_tokens) + 2,
-            _ptr(gemm_fast.status_flag(q.device)), sk, *extra, *gate_args, stream)
+            _ptr(gemm_fast.status_flag(q.device)), sk, *extra, *gate_args, *bias, stream)
         if code == _UNSUPPORTED:
             return False
         ops._check(code, "paged_attention (tcgen05 prefill, two query tiles)")
@@ -249,7 +250,7 @@ def run(q, k_pages, v_pages, block_table, out, H, G, hd, page_tokens, window, sc
         code = lib_tc.hk_attention_prefill_tc(
             _ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), int(block_table.shape[1]), _ptr(plan.items),
             plan.n_items, _ptr(out), H, G, hd, int(page_tokens), int(window), ctypes.c_float(scale * math.log2(math.e)),
-            plan.max_keys // int(page_tokens) + 2, _ptr(gemm_fast.status_flag(q.device)), sk, *extra, *gate_args, stream)
+            plan.max_keys // int(page_tokens) + 2, _ptr(gemm_fast.status_flag(q.device)), sk, *extra, *gate_args, *bias, stream)
         if code == _UNSUPPORTED:
             return False
         ops._check(code, "paged_attention (tcgen05 prefill)")
@@ -260,12 +261,12 @@ def run(q, k_pages, v_pages, block_table, out, H, G, hd, page_tokens, window, sc
             _ptr(q), _ptr(k_pages), _ptr(v_pages), ctypes.c_longlong(k_pages.shape[0]), _ptr(block_table),
             int(block_table.shape[1]), _ptr(plan.items), plan.n_items, _ptr(out), _ptr(part_o), _ptr(part_ml), H, G, hd,
             int(page_tokens), int(window), ctypes.c_float(scale * math.log2(math.e)), sk, plan.max_keys // int(page_tokens) + 2,
-            _ptr(gemm_fast.status_flag(q.device)), *extra, stream)
+            _ptr(gemm_fast.status_flag(q.device)), *extra, *bias, stream)
     if code == _UNSUPPORTED:
         code = lib.hk_attention_flash(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), int(block_table.shape[1]),
                                       _ptr(plan.items), plan.n_items, plan.nw, _ptr(out), _ptr(part_o), _ptr(part_ml), H, G, hd,
                                       int(page_tokens), int(window), ctypes.c_float(scale * math.log2(math.e)), sk,
-                                      plan.max_keys // int(page_tokens) + 2, *extra, stream)
+                                      plan.max_keys // int(page_tokens) + 2, *extra, *bias, stream)
     if code == _UNSUPPORTED:
         return False
     ops._check(code, "paged_attention (flash)")

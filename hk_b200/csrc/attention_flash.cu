@@ -43,7 +43,14 @@ struct ScoreOpts {
   float cap_log2;       // soft cap c on the scores, times log2(e): s <- c tanh(s / c); 0: none
   float cap_in;         // scale / c
   int chunk;            // a row at position p sees no key before (p / chunk) * chunk; 0: no such mask
+  const float* dist;    // [H, dist_n] in the base-2 domain: added to the score of a key n positions back, at
+  int dist_n;           //   min(n, dist_n - 1); null: none
 };
+
+// what the distance of a visible key adds to its score; `row`: the query head's part of the table
+__device__ __forceinline__ float distance_bias(const float* row, int back, const ScoreOpts& so) {
+  return __ldg(row + min(back, so.dist_n - 1));
+}
 
 // scale (and cap) a raw dot product into the base-2 exponent domain
 __device__ __forceinline__ float scaled_score(float s, float scale_log2, const ScoreOpts& so) {
@@ -116,6 +123,7 @@ attention_flash_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pa
   int row[2], pos[2], lo[2];
   bool valid[2];
   const bf16* qp[2];
+  const float* drow[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     row[i] = warp * 16 + qr + 8 * i;
@@ -126,6 +134,7 @@ attention_flash_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pa
     lo[i] = window > 0 ? max(0, pos[i] - window + 1) : 0;
     if (so.chunk > 0) lo[i] = max(lo[i], (pos[i] / so.chunk) * so.chunk);
     qp[i] = q + ((size_t)(it.q_row0 + tq) * H + g * group + row[i] % group) * HD;
+    drow[i] = so.dist ? so.dist + (size_t)(g * group + row[i] % group) * so.dist_n : nullptr;
   }
 
   // Q fragments (A operand): per k-step a0 = (r0, d 2t..), a1 = (r0+8, d 2t..), a2 = (r0, d 2t+8..), a3 = (r0+8, d 2t+8..)
@@ -209,7 +218,22 @@ attention_flash_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pa
     const int j_first = t * TILE_N, j_last = t * TILE_N + TILE_N - 1;
     const bool whole = valid[0] && valid[1] && j_first >= max(max(lo[0], lo[1]), it.kv_lo) &&
                        j_last <= min(min(pos[0], pos[1]), it.kv_hi - 1);
-    if (whole) {
+    if (whole && so.dist) {
+      // beyond the table's last distance the bias is one number per row
+      float far[2];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) far[i] = distance_bias(drow[i], so.dist_n - 1, so);
+      const bool all_far = min(pos[0], pos[1]) - j_last >= so.dist_n - 1;
+#pragma unroll
+      for (int n = 0; n < TILE_N / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = e >> 1;
+          const int j = j_first + n * 8 + 2 * qt + (e & 1);
+          s[n][e] = scaled_score(s[n][e], scale_log2, so) + (all_far ? far[i] : distance_bias(drow[i], pos[i] - j, so));
+          mt[i] = fmaxf(mt[i], s[n][e]);
+        }
+    } else if (whole) {
 #pragma unroll
       for (int n = 0; n < TILE_N / 8; ++n)
 #pragma unroll
@@ -225,7 +249,7 @@ attention_flash_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pa
           const int i = e >> 1;
           const int j = t * TILE_N + n * 8 + 2 * qt + (e & 1);
           const bool ok = valid[i] && j >= lo[i] && j <= pos[i] && j >= it.kv_lo && j < it.kv_hi;
-          s[n][e] = ok ? scaled_score(s[n][e], scale_log2, so) : -CUDART_INF_F;
+          s[n][e] = ok ? scaled_score(s[n][e], scale_log2, so) + (so.dist ? distance_bias(drow[i], pos[i] - j, so) : 0.f) : -CUDART_INF_F;
           mt[i] = fmaxf(mt[i], s[n][e]);
         }
     }
@@ -344,6 +368,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
   int row[2], pos[2], lo[2];
   bool valid[2];
   const bf16* qp[2];
+  const float* drow[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     row[i] = qr + 8 * i;
@@ -354,6 +379,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
     lo[i] = window > 0 ? max(0, pos[i] - window + 1) : 0;
     if (so.chunk > 0) lo[i] = max(lo[i], (pos[i] / so.chunk) * so.chunk);
     qp[i] = q + ((size_t)(it.q_row0 + tq) * H + g * group + row[i] % group) * HD;
+    drow[i] = so.dist ? so.dist + (size_t)(g * group + row[i] % group) * so.dist_n : nullptr;
   }
   uint32_t qf[KSTEPS][4];
 #pragma unroll
@@ -426,7 +452,7 @@ attention_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_p
         const int i = e >> 1;
         const int j = t * DT + warp * 16 + n * 8 + 2 * qt + (e & 1);
         const bool ok = valid[i] && j >= lo[i] && j <= pos[i] && j >= it.kv_lo && j < it.kv_hi;
-        s[n][e] = ok ? scaled_score(s[n][e], scale_log2, so) : -CUDART_INF_F;
+        s[n][e] = ok ? scaled_score(s[n][e], scale_log2, so) + (so.dist ? distance_bias(drow[i], pos[i] - j, so) : 0.f) : -CUDART_INF_F;
         mt[i] = fmaxf(mt[i], s[n][e]);
       }
     float corr[2], msafe[2];
@@ -646,6 +672,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
     int pos[2], lo[2];
     bool valid[2];
     const bf16* qp[2];
+    const float* drow[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       row[i] = qr + 8 * i;
@@ -656,6 +683,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       lo[i] = window > 0 ? max(0, pos[i] - window + 1) : 0;
     if (so.chunk > 0) lo[i] = max(lo[i], (pos[i] / so.chunk) * so.chunk);
       qp[i] = q + ((size_t)(it.q_row0 + tq) * H + g * group + row[i] % group) * HD;
+      drow[i] = so.dist ? so.dist + (size_t)(g * group + row[i] % group) * so.dist_n : nullptr;
     }
     uint32_t qf[KSTEPS][4];
 #pragma unroll
@@ -707,7 +735,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           const int i = e >> 1;
           const int j = t * TT + warp * 16 + nn * 8 + 2 * qt + (e & 1);
           const bool ok = valid[i] && j >= lo[i] && j <= pos[i] && j >= it.kv_lo && j < it.kv_hi;
-          s[nn][e] = ok ? scaled_score(s[nn][e], scale_log2, so) : -CUDART_INF_F;
+          s[nn][e] = ok ? scaled_score(s[nn][e], scale_log2, so) + (so.dist ? distance_bias(drow[i], pos[i] - j, so) : 0.f) : -CUDART_INF_F;
           mt[i] = fmaxf(mt[i], s[nn][e]);
         }
       float corr[2], msafe[2];
@@ -912,8 +940,8 @@ int launch_hd(int nw, const void* q, const void* kp, const void* vp, const int* 
   return HK_ERR_UNSUPPORTED;
 }
 
-ScoreOpts make_opts(int sink, const float* sinks, float softcap, float scale_log2, int chunk) {
-  ScoreOpts so = {sink, sink ? sinks : nullptr, 0.f, 0.f, chunk > 0 ? chunk : 0};
+ScoreOpts make_opts(int sink, const float* sinks, float softcap, float scale_log2, int chunk, const float* dist = nullptr, int dist_n = 0) {
+  ScoreOpts so = {sink, sink ? sinks : nullptr, 0.f, 0.f, chunk > 0 ? chunk : 0, dist_n > 0 ? dist : nullptr, dist_n};
   if (softcap > 0.f) {
     so.cap_log2 = softcap * 1.4426950408889634f;
     so.cap_in = scale_log2 / so.cap_log2;       // scale / softcap
@@ -928,13 +956,14 @@ ScoreOpts make_opts(int sink, const float* sinks, float softcap, float scale_log
 // (16 * nw) / (H / G) query tokens.  part_o [parts, G, 16*nw, hd] and part_ml [parts, G, 16*nw, 2] are
 // fp32 scratch for items with part >= 0.  scale_log2 = scale * log2(e).  pages_cap: the most pages any item's key
 // range spans (the decode variant keeps that many page ids in shared memory).  sink, sinks, softcap, chunk: see
-// `ScoreOpts` (sinks: one score per query head or null; softcap and chunk 0 for none).
+// `ScoreOpts` (sinks: one score per query head or null; softcap and chunk 0 for none; dist [H, dist_n], times log2(e)
+// already, or null).
 HK_API int hk_attention_flash(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                               int table_stride, const void* items, int n_items, int nw, void* out, float* part_o,
                               float* part_ml, int H, int G, int hd, int page_tokens, int window, float scale_log2, int sink,
-                              int pages_cap, const float* sinks, float softcap, int chunk, void* stream) {
+                              int pages_cap, const float* sinks, float softcap, int chunk, const float* dist, int dist_n, void* stream) {
   if (n_items <= 0) return 0;
-  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk);
+  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk, dist, dist_n);
   if (G < 1 || H % G != 0 || (H / G) > 16 * nw || G > 65535) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
 #define HK_HD(D) \
@@ -1014,9 +1043,9 @@ HK_API int hk_attention_decode_tma(const void* q, const void* k_pages, const voi
                                    const int* block_table, int table_stride, const void* items, int n_items, void* out,
                                    float* part_o, float* part_ml, int H, int G, int hd, int page_tokens, int window,
                                    float scale_log2, int sink, int pages_cap, int* status, const float* sinks, float softcap,
-                                   int chunk, void* stream) {
+                                   int chunk, const float* dist, int dist_n, void* stream) {
   if (n_items <= 0) return 0;
-  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk);
+  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk, dist, dist_n);
   if (G < 1 || H % G != 0 || (H / G) > 16 || G > 65535) return HK_ERR_UNSUPPORTED;
   if ((hd != 64 && hd != 128) || page_tokens < 16 || (page_tokens & (page_tokens - 1))) return HK_ERR_UNSUPPORTED;
   if (((uintptr_t)k_pages & 127) || ((uintptr_t)v_pages & 127)) return HK_ERR_UNSUPPORTED;
@@ -1074,7 +1103,7 @@ HK_API int hk_attention_decode_noalloc(const void* q, const void* k_pages, const
   float* part_o = scratch;
   float* part_ml = scratch + (size_t)n_parts * G * rows * hd;
   int code = hk_attention_flash(q, k_pages, v_pages, block_table, table_stride, items, n_items, 1, out, part_o, part_ml, H, G,
-                                hd, page_tokens, window, scale_log2, 0, pages_cap, nullptr, 0.f, 0, stream);
+                                hd, page_tokens, window, scale_log2, 0, pages_cap, nullptr, 0.f, 0, nullptr, 0, stream);
   if (code != 0 || n_parts == 0) return code;
   return hk_attention_combine(part_o, part_ml, first, count, row0, out, n_tokens, H, G, hd, (int)rows, 0, nullptr, stream);
 }

@@ -17,6 +17,8 @@
 //   v_stride    elements between the values of consecutive tokens of a page; when it is not vd the values lie inside
 //               wider rows: a cache that keeps ONE tensor per token whose first vd dims are the value (v_pages = k_pages,
 //               v_stride = hd);
+//   dist        float [H, dist_n]: the score of a key n positions back is raised by dist[h, min(n, dist_n - 1)] (behind the
+//               scale and the cap; a bias learned per distance, the last entry standing for all further ones);
 //   gate        fp32 logits [n, gate_ld >= H * vd]: the output is multiplied by gate_scale * sigmoid(gate[t, h * vd + d]).
 //
 // Reference counterpart: `attention`, src/cuda_device.zig:1494-1594 (block per (token, head),
@@ -35,6 +37,8 @@ struct AgOptions {
   const float* gate;
   long long gate_ld;
   float gate_scale;
+  const float* dist;
+  int dist_n;
 };
 
 // AG_MAX_PER_LANE: dims per lane, 8 for widths up to 256, 20 up to 640
@@ -82,6 +86,7 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
     }
     s = warp_sum(s);
     if (cap > 0.f) s = cap * tanhf(s * inv_cap);
+    if (opt.dist) s += opt.dist[(size_t)h * opt.dist_n + min(pos - j, opt.dist_n - 1)];
     float mn = fmaxf(m, s);
     float corr = expf(m - mn);
     float p = expf(s - mn);
@@ -141,12 +146,15 @@ HK_API int hk_attention_generic(const void* q, const void* k_pages, const void* 
                                 const int* block_table, int table_stride, const int* positions,
                                 const int* slot_of_token, void* out, int n, int H, int G, int hd,
                                 int page_tokens, int window, float scale, int vd, int sink, const float* sinks, float softcap,
-                                int chunk, int v_stride, const float* gate, long long gate_ld, float gate_scale, void* stream) {
+                                int chunk, int v_stride, const float* gate, long long gate_ld, float gate_scale, const float* dist,
+                                int dist_n, void* stream) {
   if (n <= 0) return 0;
   const int widest = hd > vd ? hd : vd;
-  if (widest > 640 || hd < 1 || G < 1 || H % G != 0 || vd < 1 || v_stride < vd || softcap < 0.f || chunk < 0) return HK_ERR_UNSUPPORTED;
+  if (widest > 640 || hd < 1 || G < 1 || H % G != 0 || vd < 1 || v_stride < vd || softcap < 0.f || chunk < 0 ||
+      (dist && dist_n < 1))
+    return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
-  AgOptions opt = {softcap, chunk, v_stride, sinks, gate, gate_ld, gate_scale};
+  AgOptions opt = {softcap, chunk, v_stride, sinks, gate, gate_ld, gate_scale, dist, dist_n};
   if (dtype != HK_F32 && dtype != HK_BF16) return HK_ERR_UNSUPPORTED;
 #define AG_GO(T, PER) ag_launch<T, PER>(q, k_pages, v_pages, block_table, table_stride, positions, slot_of_token, out, n, H, G, hd, \
                                         page_tokens, window, scale, vd, sink, opt, s)

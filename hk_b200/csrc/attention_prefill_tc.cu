@@ -56,6 +56,8 @@ struct ScoreOpts {
   const float* gate;    // output gate's logits, float32 [tokens, gate_ld >= H * HD] (16-byte aligned rows), or null:
   long long gate_ld;    //   out[t, h, d] is multiplied by gate_scale * sigmoid(gate[t, h * HD + d]) before it is rounded
   float gate_scale;
+  const float* dist;    // [H, dist_n] in the base-2 domain: added to the score of a key n positions back, at
+  int dist_n;           //   min(n, dist_n - 1); null: none
 };
 
 // eight values of a row of O, normalised and (with a gate) gated, packed into bfloat16
@@ -90,6 +92,15 @@ __device__ __forceinline__ uint32_t capped_score(uint32_t raw, const ScoreOpts& 
   return raw == 0xff800000u ? raw : __float_as_uint(fmaf(-2.0f * so.cap_log2, r, so.cap_log2));
 }
 
+// Raw scores (or -inf) of N neighbouring keys from key j0 on into the base-2 exponent domain with the bias of each key's
+// distance; `row`: the query head's part of the table.  (Keys behind the query are masked: their distance only has to
+// stay inside the table.)
+template <int N>
+__device__ __forceinline__ void add_distance_bias(uint32_t* su, const float* row, int back0, float sl, int dist_n) {
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+    su[i] = __float_as_uint(fmaf(__uint_as_float(su[i]), sl, __ldg(row + min(max(back0 - i, 0), dist_n - 1))));
+}
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void mbar_init(uint64_t* bar, uint32_t count) {
@@ -420,6 +431,8 @@ attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__
     const float sl = so.cap_log2 > 0.f ? 1.0f : scale_log2;      // capped scores are in the exponent's domain already
     const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
     constexpr int HK = TK / 2, HO = HD / 2;          // keys and O columns per thread
+    const float* drow = so.dist ? so.dist + (size_t)(g * group + (valid ? r % group : 0)) * so.dist_n : nullptr;
+    const float far_bias = drow ? drow[so.dist_n - 1] : 0.f;
     float m = -CUDART_INF_F, l = 0.f;
     bool ok = true;
     for (int t = t_begin; t < t_end; ++t) {
@@ -449,12 +462,22 @@ attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__
         for (int i = 0; i < HK; ++i) su[i] = capped_score(su[i], so);
       }
       float mraw = -CUDART_INF_F;
+      // The two threads of a row compare maxima in the exponent's domain.  Where all of this thread's keys are further back
+      // than the table reaches, their bias is one number and rides on the maximum and the exponent's constant; else every
+      // score takes its own.
+      float slt = sl, add = far_bias;
+      if (drow && pos - (j0 + HK - 1) < so.dist_n - 1) {
+        add_distance_bias<HK>(su, drow, pos - j0, sl, so.dist_n);
+        slt = 1.0f;
+        add = 0.f;
+      }
 #pragma unroll
       for (int i = 0; i < HK; ++i) mraw = fmaxf(mraw, __uint_as_float(su[i]));
+      mraw = fmaf(mraw, slt, add);
       sm.xmax[n & 1][half][r] = mraw;
       asm volatile("bar.sync %0, 64;" ::"r"(1 + quarter) : "memory");     // the two warps of this quarter
       mraw = fmaxf(mraw, sm.xmax[n & 1][half ^ 1][r]);
-      const float mt = mraw * sl;
+      const float mt = mraw;
       // Lazy rescaling: the exponentials are taken against a reference maximum `m` that only moves when the row's
       // true maximum has run ahead of it by more than 2^8 (P then stays below 256, exact in bf16's range, and
       // sum and O stay consistent with it, so the result is the same).  Moving it costs a pass over the O row
@@ -475,8 +498,8 @@ attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__
       uint32_t pw[HK / 2];
 #pragma unroll
       for (int e = 0; e < HK / 2; ++e) {
-        const float p0 = ex2(fmaf(__uint_as_float(su[2 * e]), sl, -msafe));
-        const float p1 = ex2(fmaf(__uint_as_float(su[2 * e + 1]), sl, -msafe));
+        const float p0 = ex2(fmaf(__uint_as_float(su[2 * e]), slt, add - msafe));
+        const float p1 = ex2(fmaf(__uint_as_float(su[2 * e + 1]), slt, add - msafe));
         l += p0 + p1;
         __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
         pw[e] = *reinterpret_cast<uint32_t*>(&pk);
@@ -768,6 +791,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
     cp_async_wait<0>();
     fence_async_proxy();
     mbar_arrive(&sm.q_full);
+    const float* drow = so.dist ? so.dist + (size_t)(g * group + (valid ? row % group : 0)) * so.dist_n : nullptr;
+    const float far_bias = drow ? drow[so.dist_n - 1] : 0.f;
     float m = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
     bool ok = true;
     if (qt == 0 || two) {
@@ -802,13 +827,20 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
 #pragma unroll
             for (int i = 0; i < 32; ++i) su[i] = capped_score(su[i], so);
           }
+          // keys further back than the table reaches share one bias, which rides on the exponent's constant
+          float slt = sl, add = far_bias;
+          if (drow && pos - (j0 + 32 * c + 31) < so.dist_n - 1) {
+            add_distance_bias<32>(su, drow, pos - (j0 + 32 * c), sl, so.dist_n);
+            slt = 1.0f;
+            add = 0.f;
+          }
           float mx[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) mx[e] = fmaxf(mx[e], fmaxf(__uint_as_float(su[i + 2 * e]), __uint_as_float(su[i + 2 * e + 1])));
           }
-          const float cm = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * sl;
+          const float cm = fmaf(fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])), slt, add);
           const bool move = cm > m + 8.0f;
           if (__any_sync(0xffffffffu, move)) {
             const float mn = move ? ceilf(cm) : m;
@@ -843,12 +875,12 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
             }
             m = mn;
           }
-          const float msafe = m == -CUDART_INF_F ? 0.f : m;
+          const float shift = add - (m == -CUDART_INF_F ? 0.f : m);
           uint32_t pw[16];
 #pragma unroll
           for (int e = 0; e < 16; ++e) {
-            const float p0 = ex2(fmaf(__uint_as_float(su[2 * e]), sl, -msafe));
-            const float p1 = ex2(fmaf(__uint_as_float(su[2 * e + 1]), sl, -msafe));
+            const float p0 = ex2(fmaf(__uint_as_float(su[2 * e]), slt, shift));
+            const float p1 = ex2(fmaf(__uint_as_float(su[2 * e + 1]), slt, shift));
             l0 += p0;
             l1 += p1;
             __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
@@ -936,8 +968,9 @@ int launch2(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, const i
 }
 
 ScoreOpts make_opts(int sink, const float* sinks, float softcap, float scale_log2, int chunk, const float* gate, long long gate_ld,
-                    float gate_scale) {
-  ScoreOpts so = {sink, sink ? sinks : nullptr, 0.f, 0.f, chunk > 0 ? chunk : 0, gate, gate_ld, gate_scale};
+                    float gate_scale, const float* dist, int dist_n) {
+  ScoreOpts so = {sink, sink ? sinks : nullptr, 0.f, 0.f, chunk > 0 ? chunk : 0, gate, gate_ld, gate_scale, dist_n > 0 ? dist : nullptr,
+                  dist_n};
   if (softcap > 0.f) {
     so.cap_log2 = softcap * 1.4426950408889634f;
     so.cap_in2 = 2.8853900817779268f * scale_log2 / so.cap_log2;       // 2 log2(e) scale / softcap
@@ -953,14 +986,15 @@ ScoreOpts make_opts(int sink, const float* sinks, float softcap, float scale_log
 // other than 64 and 128 and groups above 128 heads.  sink, sinks, softcap, chunk: see `ScoreOpts` (sinks: one score per
 // query head or null; softcap and chunk 0 for none).  gate (float32 logits [tokens, gate_ld], 16-byte aligned, gate_ld a
 // multiple of 4; or null): the result is multiplied by gate_scale * sigmoid(gate[t, h * hd + d]) before it is rounded.
+// dist: see `ScoreOpts` (or null).
 HK_API int hk_attention_prefill_tc(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                                    int table_stride, const void* items, int n_items, void* out, int H, int G, int hd,
                                    int page_tokens, int window, float scale_log2, int pages_cap, int* status, int sink,
                                    const float* sinks, float softcap, int chunk, const float* gate, long long gate_ld,
-                                   float gate_scale, void* stream) {
+                                   float gate_scale, const float* dist, int dist_n, void* stream) {
   if (n_items <= 0) return 0;
   if (gate != nullptr && ((((uintptr_t)gate) & 15) != 0 || (gate_ld & 3) != 0 || gate_ld < (long long)H * hd)) return HK_ERR_UNSUPPORTED;
-  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk, gate, gate_ld, gate_scale);
+  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk, gate, gate_ld, gate_scale, dist, dist_n);
   if (G < 1 || H % G != 0 || (H / G) > ROWS || G > 65535 || page_tokens < 1 || !(scale_log2 > 0.f)) return HK_ERR_UNSUPPORTED;
   if ((((uintptr_t)q | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)out) & 15) != 0) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
@@ -976,10 +1010,10 @@ HK_API int hk_attention_prefill_tc2(const void* q, const void* k_pages, const vo
                                     const int* block_table, int table_stride, const void* items, int n_items, void* out, int H,
                                     int G, int hd, int page_tokens, int window, float scale_log2, int pages_cap, int* status,
                                     int sink, const float* sinks, float softcap, int chunk, const float* gate, long long gate_ld,
-                                    float gate_scale, void* stream) {
+                                    float gate_scale, const float* dist, int dist_n, void* stream) {
   if (n_items <= 0) return 0;
   if (gate != nullptr && ((((uintptr_t)gate) & 15) != 0 || (gate_ld & 3) != 0 || gate_ld < (long long)H * hd)) return HK_ERR_UNSUPPORTED;
-  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk, gate, gate_ld, gate_scale);
+  const ScoreOpts so = make_opts(sink, sinks, softcap, scale_log2, chunk, gate, gate_ld, gate_scale, dist, dist_n);
   if (G < 1 || H % G != 0 || (H / G) > ROWS || G > 65535 || page_tokens < 1 || !(scale_log2 > 0.f)) return HK_ERR_UNSUPPORTED;
   if (hd != 64 && hd != 128) return HK_ERR_UNSUPPORTED;
   const bool boxes_ok = (page_tokens % 8 == 0 && TK % page_tokens == 0) || page_tokens % TK == 0;

@@ -232,6 +232,16 @@ HK_API int hk_rms_norm(const float* x, const float* w, const int* rows, void* ou
 // `norm_after` = 1 moves the per-head norm behind the rotation, where a null weight means a weight of ones
 // (x over its root mean square).  `tied_v` = 1: the projection has no v heads (a row holds H + G heads) and a
 // token's value is its key as projected, before rotation and norm, of which the first `vd` dims are kept.
+// `qt` (coef, every): a query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) before it is stored
+// (every 0: not at all).
+struct QueryFactor {
+  float coef;
+  int every;
+};
+__device__ __forceinline__ float query_factor(const QueryFactor& qt, int pos) {
+  return qt.every > 0 ? fmaf(qt.coef, logf((float)((pos + 1) / qt.every) + 1.0f), 1.0f) : 1.0f;
+}
+
 #define QKR_MAX_HD 256
 #define QKR_WARPS 4
 
@@ -242,7 +252,8 @@ __global__ void qk_norm_rope_kv_write_kernel(
     const float* __restrict__ sin_t, int rot, const int* __restrict__ positions,
     const int* __restrict__ slot_of_token, const int* __restrict__ block_table, int table_stride,
     T* __restrict__ k_pages, T* __restrict__ v_pages, int n, int H, int G, int hd, int page_tokens,
-    int write_kv, const float* __restrict__ bias, int pairing, int norm_after, int tied_v, int vd, long long ld) {
+    int write_kv, const float* __restrict__ bias, int pairing, int norm_after, int tied_v, int vd, long long ld,
+    QueryFactor qt) {
   __shared__ float buf[QKR_WARPS][QKR_MAX_HD];
   pdl_launch_dependents();
   pdl_wait();
@@ -310,6 +321,11 @@ __global__ void qk_norm_rope_kv_write_kernel(
   }
   T* dst;
   int width = hd;
+  if (kind == 0 && qt.every > 0) {
+    const float f = query_factor(qt, pos);
+    for (int i = lane; i < hd; i += 32) v[i] *= f;      // a lane's own entries
+    __syncwarp();
+  }
   if (kind == 0) {
     dst = q_out + (size_t)t * H * hd + (size_t)hh * hd;
   } else if (kind == 1) {
@@ -333,7 +349,8 @@ qk_norm_rope_kv_write_vec_kernel(
     const float* __restrict__ sin_t, int rot, const int* __restrict__ positions,
     const int* __restrict__ slot_of_token, const int* __restrict__ block_table, int table_stride,
     T* __restrict__ k_pages, T* __restrict__ v_pages, int n, int H, int G, int hd, int page_tokens,
-    int write_kv, const float* __restrict__ bias, int pairing, int norm_after, int tied_v, int vd, long long ld) {
+    int write_kv, const float* __restrict__ bias, int pairing, int norm_after, int tied_v, int vd, long long ld,
+    QueryFactor qt) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5;
@@ -419,6 +436,10 @@ qk_norm_rope_kv_write_vec_kernel(
   }
   if (!active || page < 0) return;
   T* dst;
+  if (kind == 0 && qt.every > 0) {
+    const float f = query_factor(qt, pos);
+    v = make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
+  }
   if (kind == 0) {
     dst = q_out + (size_t)t * H * hd + (size_t)hh * hd;
   } else if (kind == 1) {
@@ -441,7 +462,9 @@ HK_API int hk_qk_norm_rope_kv_write(const float* qkv, void* q_out, int dtype, co
                                     const int* block_table, int table_stride, void* k_pages,
                                     void* v_pages, int n, int H, int G, int hd, int page_tokens,
                                     int write_kv, const float* bias, int pairing, int norm_after, int tied_v, int vd,
-                                    long long ld, void* stream) {
+                                    long long ld, float qt_coef, int qt_every, void* stream) {
+  const QueryFactor qt = {qt_coef, qt_every};
+  if (qt_every < 0) return HK_ERR_UNSUPPORTED;
   if (ld <= 0) ld = (long long)(H + G) * hd + (tied_v ? 0 : (long long)G * vd);
   if (n <= 0) return 0;
   if (hd > QKR_MAX_HD || hd < 2 || rot > hd || (rot & 1) || pairing < 0 || pairing > 1) return HK_ERR_UNSUPPORTED;
@@ -455,23 +478,160 @@ HK_API int hk_qk_norm_rope_kv_write(const float* qkv, void* q_out, int dtype, co
     if (dtype == HK_F32)
       return hk_launch_pdl(qk_norm_rope_kv_write_vec_kernel<float>, dim3(vblocks), dim3(QKV_WARPS * 32), 0, s, qkv, (float*)q_out,
                        q_w, k_w, eps, cos_t, sin_t, rot, positions, slot_of_token, block_table, table_stride, (float*)k_pages,
-                       (float*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld);
+                       (float*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld, qt);
     if (dtype == HK_BF16)
       return hk_launch_pdl(qk_norm_rope_kv_write_vec_kernel<bf16>, dim3(vblocks), dim3(QKV_WARPS * 32), 0, s, qkv, (bf16*)q_out, q_w,
                        k_w, eps, cos_t, sin_t, rot, positions, slot_of_token, block_table, table_stride, (bf16*)k_pages,
-                       (bf16*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld);
+                       (bf16*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld, qt);
     return HK_ERR_UNSUPPORTED;
   }
   unsigned blocks = (unsigned)((items + QKR_WARPS - 1) / QKR_WARPS);
   if (dtype == HK_F32)
     return hk_launch(qk_norm_rope_kv_write_kernel<float>, dim3(blocks), dim3(QKR_WARPS * 32), 0, s, qkv, (float*)q_out, q_w,
                          k_w, eps, cos_t, sin_t, rot, positions, slot_of_token, block_table, table_stride, (float*)k_pages,
-                         (float*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld);
+                         (float*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld, qt);
   if (dtype == HK_BF16)
     return hk_launch(qk_norm_rope_kv_write_kernel<bf16>, dim3(blocks), dim3(QKR_WARPS * 32), 0, s, qkv, (bf16*)q_out, q_w,
                          k_w, eps, cos_t, sin_t, rot, positions, slot_of_token, block_table, table_stride, (bf16*)k_pages,
-                         (bf16*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld);
+                         (bf16*)v_pages, n, H, G, hd, page_tokens, write_kv, bias, pairing, norm_after, tied_v, vd, ld, qt);
   return HK_ERR_UNSUPPORTED;
+}
+
+// ------------------------------------------------- norm over the whole projection + cache write
+// A CTA per token of the projection row qkv[t] = [q: H hd | k: G hd | v: G vd] (fp32, rows ld floats apart): `bias` (or
+// null) is added, then q is divided by the root mean square of ALL its rows together (over q_count numbers: heads may be
+// filled up with zeros to a width of their own, which the mean does not count), k likewise over k_count, times weights of
+// the rows' width; q then times its factor by position and to q_out[n, H hd], k and v into the token's cache page.  The row
+// stays in shared memory between the two passes.  V: numbers a thread moves at once.
+#define RNW_THREADS 256
+template <typename T, int V>
+__global__ void __launch_bounds__(RNW_THREADS)
+qk_row_norm_kv_write_kernel(const float* __restrict__ qkv, long long ld, const float* __restrict__ bias, T* __restrict__ q_out,
+                            const float* __restrict__ q_w, const float* __restrict__ k_w, float q_count, float k_count, float eps,
+                            const int* __restrict__ positions, const int* __restrict__ slot_of_token, const int* __restrict__ block_table,
+                            int table_stride, T* __restrict__ k_pages, T* __restrict__ v_pages, int H, int G, int hd, int vd,
+                            int page_tokens, int write_kv, QueryFactor qt) {
+  extern __shared__ __align__(16) float rowv[];       // [QW + KW]
+  __shared__ float part[2][RNW_THREADS / 32];
+  const int t = blockIdx.x, QW = H * hd, KW = G * hd, VW = G * vd;
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* src = qkv + (size_t)t * ld;
+  const int pos = positions[t];
+  int page = -1;
+  if (write_kv) page = block_table[(size_t)slot_of_token[t] * table_stride + pos / page_tokens];
+  const int place = pos % page_tokens;
+  auto load = [&](int i, float* f) {
+    if (V == 4) {
+      float4 a = *reinterpret_cast<const float4*>(src + i);
+      if (bias) {
+        const float4 b = *reinterpret_cast<const float4*>(bias + i);
+        a = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+      }
+      *reinterpret_cast<float4*>(f) = a;
+    } else {
+      f[0] = src[i] + (bias ? bias[i] : 0.f);
+    }
+  };
+  auto store = [&](T* dst, const float* f) {
+    if (V == 4 && sizeof(T) == 2) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
+      *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    } else if (V == 4) {
+      *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(f);
+    } else {
+      dst[0] = from_f32<T>(f[0]);
+    }
+  };
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x * V; i < QW + KW; i += RNW_THREADS * V) {
+    float f[4];
+    load(i, f);
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      rowv[i + e] = f[e];
+      if (i < QW) sq = fmaf(f[e], f[e], sq); else sk = fmaf(f[e], f[e], sk);
+    }
+  }
+  if (page >= 0)                                      // (a page below 0 is never scheduled by the host)
+    for (int i = threadIdx.x * V; i < VW; i += RNW_THREADS * V) {
+      float f[4];
+      load(QW + KW + i, f);
+      store(v_pages + (((size_t)page * G + i / vd) * page_tokens + place) * vd + i % vd, f);
+    }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) {
+    part[0][threadIdx.x >> 5] = sq;
+    part[1][threadIdx.x >> 5] = sk;
+  }
+  __syncthreads();
+  float tq = 0.f, tk = 0.f;
+#pragma unroll
+  for (int i = 0; i < RNW_THREADS / 32; ++i) {
+    tq += part[0][i];
+    tk += part[1][i];
+  }
+  const float iq = 1.0f / sqrtf(tq / q_count + eps), ik = 1.0f / sqrtf(tk / k_count + eps), factor = query_factor(qt, pos);
+  for (int i = threadIdx.x * V; i < QW + KW; i += RNW_THREADS * V) {
+    float f[4];
+#pragma unroll
+    for (int e = 0; e < V; ++e) f[e] = i < QW ? rowv[i + e] * iq * q_w[i + e] * factor : rowv[i + e] * ik * k_w[i - QW + e];
+    if (i < QW) {
+      store(q_out + (size_t)t * QW + i, f);
+    } else if (page >= 0) {
+      const int c = i - QW;
+      store(k_pages + (((size_t)page * G + c / hd) * page_tokens + place) * hd + c % hd, f);
+    }
+  }
+}
+
+HK_API int hk_qk_row_norm_kv_write(const float* qkv, long long ld, const float* bias, void* q_out, int dtype, const float* q_w,
+                                   const float* k_w, float q_count, float k_count, float eps, const int* positions,
+                                   const int* slot_of_token, const int* block_table, int table_stride, void* k_pages, void* v_pages,
+                                   int n, int H, int G, int hd, int vd, int page_tokens, int write_kv, float qt_coef, int qt_every,
+                                   void* stream) {
+  if (n <= 0) return 0;
+  if (H < 1 || G < 1 || hd < 1 || vd < 1 || page_tokens < 1 || qt_every < 0) return HK_ERR_UNSUPPORTED;
+  const QueryFactor qt = {qt_coef, qt_every};
+  const size_t smem = (size_t)(H + G) * hd * sizeof(float);
+  if (smem > 200 * 1024) return HK_ERR_UNSUPPORTED;
+  const uintptr_t all = (uintptr_t)qkv | (uintptr_t)bias | (uintptr_t)q_out | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)k_pages | (uintptr_t)v_pages;
+  const bool vec = (hd & 3) == 0 && (vd & 3) == 0 && (ld & 3) == 0 && (all & 15) == 0;
+  cudaStream_t s = (cudaStream_t)stream;
+#define RNW_GO(T, V)                                                                                                             \
+  do {                                                                                                                           \
+    static HkSmemCache cache;                                                                                                    \
+    if (int e = hk_allow_smem(qk_row_norm_kv_write_kernel<T, V>, smem, cache)) return e;                                         \
+    return hk_launch_pdl(qk_row_norm_kv_write_kernel<T, V>, dim3(n), dim3(RNW_THREADS), smem, s, qkv, ld, bias, (T*)q_out, q_w, k_w, \
+                         q_count, k_count, eps, positions, slot_of_token, block_table, table_stride, (T*)k_pages, (T*)v_pages, H, G, hd, \
+                         vd, page_tokens, write_kv, qt);                                                                         \
+  } while (0)
+  if (dtype == HK_F32) {
+    if (vec) RNW_GO(float, 4);
+    RNW_GO(float, 1);
+  }
+  if (dtype == HK_BF16) {
+    if (vec) RNW_GO(bf16, 4);
+    RNW_GO(bf16, 1);
+  }
+#undef RNW_GO
+  return HK_ERR_UNSUPPORTED;
+}
+
+// ----------------------------------------------------------------------------- soft cap
+// x <- cap * tanh(x / cap) in place.
+__global__ void soft_cap_kernel(float* __restrict__ x, long long total, float cap, float inv_cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < total) x[i] = cap * tanhf(x[i] * inv_cap);
+}
+
+HK_API int hk_soft_cap(float* x, long long total, float cap, void* stream) {
+  if (total <= 0) return 0;
+  if (!(cap > 0.f)) return HK_ERR_UNSUPPORTED;
+  return hk_launch_pdl(soft_cap_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, (cudaStream_t)stream, x, total, cap, 1.0f / cap);
 }
 
 // ----------------------------------------------------------------------------- bias

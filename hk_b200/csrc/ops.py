@@ -157,6 +157,59 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tenso
                            ctypes.c_longlong(ldx), ctypes.c_float(eps), _stream()), "rms_norm")
 
 
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor,
+               rows: Optional[torch.Tensor] = None) -> None:
+    """out[r, :] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias of row rows[r] (or r) of x (float32)."""
+    _need(x, "x", torch.float32, 2)
+    _need(weight, "weight", torch.float32, 1)
+    _need(bias, "bias", torch.float32, 1)
+    _need(out, "out", dims=2)
+    d, n_out = x.shape[1], out.shape[0]
+    if weight.shape[0] != d or bias.shape[0] != d or out.shape[1] != d:
+        raise KernelError("layer_norm: widths of x, weight, bias and out differ")
+    if rows is None:
+        if n_out != x.shape[0]:
+            raise KernelError("layer_norm: out has other rows than x")
+    else:
+        _need(rows, "rows", torch.int32, 1)
+        if rows.shape[0] < n_out:
+            raise KernelError("layer_norm: fewer row indices than output rows")
+    lib = build.load("norms")
+    _check(lib.hk_layer_norm(_ptr(x), _ptr(weight), _ptr(bias), _ptr(rows), _ptr(out), _dt(out), n_out, d, ctypes.c_float(eps),
+                             _stream()), "layer_norm")
+
+
+def pair_norm_add(a, wa, eps_a: float, scale_a: float, b, wb, eps_b: float, scale_b: float, residual, a_bias=None,
+                  accumulate: bool = True, next_norm=None, next_out=None) -> None:
+    """residual[r, :] (+)= scale_a * N(a + a_bias) * wa + scale_b * N(b) * wb with N(y) = y / sqrt(mean(y^2) + eps) over the row
+    (all float32; a_bias [d] or None).  `next_norm` (weight, bias, eps): the new residual row's layer norm goes to `next_out`
+    in the same pass."""
+    for name, t in (("a", a), ("b", b), ("residual", residual)):
+        _need(t, name, torch.float32, 2)
+        if t.shape != residual.shape:
+            raise KernelError("pair_norm_add: a, b and residual must have one shape")
+    n, d = residual.shape
+    for name, t in (("wa", wa), ("wb", wb), ("a_bias", a_bias)):
+        if t is not None:
+            _need(t, name, torch.float32, 1)
+            if t.shape[0] != d:
+                raise KernelError(f"pair_norm_add: {name} must have one entry per column")
+    lw = lb = None
+    leps = 0.0
+    if next_norm is not None:
+        lw, lb, leps = next_norm
+        _need(lw, "next_norm weight", torch.float32, 1)
+        _need(lb, "next_norm bias", torch.float32, 1)
+        _need(next_out, "next_out", dims=2)
+        if lw.shape[0] != d or lb.shape[0] != d or next_out.shape != residual.shape:
+            raise KernelError("pair_norm_add: the next norm does not fit")
+    lib = build.load("norms")
+    _check(lib.hk_pair_norm_add(_ptr(a), _ptr(a_bias), _ptr(wa), ctypes.c_float(eps_a), ctypes.c_float(scale_a), _ptr(b), _ptr(wb),
+                                ctypes.c_float(eps_b), ctypes.c_float(scale_b), _ptr(residual), 1 if accumulate else 0, _ptr(lw),
+                                _ptr(lb), ctypes.c_float(leps), _ptr(next_out if lw is not None else None),
+                                _dt(next_out) if lw is not None else F32, n, d, _stream()), "pair_norm_add")
+
+
 # ---- swiglu ---------------------------------------------------------------------------
 
 
@@ -258,7 +311,8 @@ PAIRINGS = {"half": 0, "adjacent": 1}
 
 def qk_norm_rope_kv_write(qkv, q_out, q_weight, k_weight, eps, cos, sin, rotary_dim, positions,
                           slot_of_token, block_table, k_pages, v_pages, n_heads, n_kv_heads, head_dim,
-                          page_tokens, write_kv=True, bias=None, pairing="half", norm_after=False, tied_v=False) -> None:
+                          page_tokens, write_kv=True, bias=None, pairing="half", norm_after=False, tied_v=False,
+                          q_factor=None) -> None:
     """Splits the fused projection qkv[n, (H+G)*hd + G*vd] (float32; vd = v_pages' width, hd unless the values have a
     width of their own): q heads are normalised (if
     q_weight), rotated (if rotary_dim > 0) and stored to q_out[n, H*hd]; k heads likewise and
@@ -266,7 +320,8 @@ def qk_norm_rope_kv_write(qkv, q_out, q_weight, k_weight, eps, cos, sin, rotary_
     `bias` (float32 [(H+2G)*hd]) is added to the projection first.  `pairing`: "half" rotates dims
     (i, i + rotary_dim/2), "adjacent" dims (2i, 2i+1).  `norm_after`: the per-head norm comes behind the
     rotation, and a missing weight then means a weight of ones.  `tied_v`: qkv is [n, (H+G)*hd] and a token's
-    value is its key as projected (before norm and rotation), of which the first v_pages.shape[-1] dims are kept."""
+    value is its key as projected (before norm and rotation), of which the first v_pages.shape[-1] dims are kept.
+    `q_factor` (coef, every): a query at position p is then multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
     if pairing not in PAIRINGS:
         raise KernelError(f"qk_norm_rope_kv_write: pairing {pairing!r} is neither 'half' nor 'adjacent'")
     if not isinstance(qkv, torch.Tensor) or not qkv.is_cuda or qkv.dtype != torch.float32 or qkv.dim() != 2 or qkv.stride(1) != 1:
@@ -310,8 +365,53 @@ def qk_norm_rope_kv_write(qkv, q_out, q_weight, k_weight, eps, cos, sin, rotary_
         _ptr(positions), _ptr(slot_of_token), _ptr(block_table if write_kv else None),
         int(block_table.shape[1]) if write_kv else 0, _ptr(k_pages if write_kv else None),
         _ptr(v_pages if write_kv else None), n, H, G, hd, int(page_tokens), 1 if write_kv else 0, _ptr(bias),
-        PAIRINGS[pairing], 1 if norm_after else 0, 1 if tied_v else 0, vd, ctypes.c_longlong(qkv.stride(0)), _stream()),
+        PAIRINGS[pairing], 1 if norm_after else 0, 1 if tied_v else 0, vd, ctypes.c_longlong(qkv.stride(0)),
+        *_query_factor(q_factor), _stream()),
         "qk_norm_rope_kv_write")
+
+
+def _query_factor(q_factor):
+    coef, every = q_factor if q_factor is not None else (0.0, 0)
+    if q_factor is not None and int(every) < 1:
+        raise KernelError("the queries' factor needs a positive number of positions per step")
+    return ctypes.c_float(coef), int(every)
+
+
+def qk_row_norm_kv_write(qkv, q_out, q_weight, k_weight, q_count: int, k_count: int, eps: float, positions, slot_of_token, block_table,
+                         k_pages, v_pages, n_heads: int, n_kv_heads: int, head_dim: int, page_tokens: int, write_kv: bool = True,
+                         bias=None, q_factor=None) -> None:
+    """For an attention that norms q and k over the whole projection: splits the float32 row qkv[n, (H+G)*hd + G*vd] (a column
+    slice; + bias), divides all of q together by its root mean square (the sum of squares over q_count, so that columns of
+    zeros that fill heads up do not count; eps inside the root), k likewise over k_count, times q_weight [H*hd] and k_weight
+    [G*hd]; q, times its factor by position (`q_factor` as in `qk_norm_rope_kv_write`), goes to q_out[n, H*hd], k and v to the
+    token's place in the cache pages."""
+    H, G, hd = n_heads, n_kv_heads, head_dim
+    _need(q_out, "q_out", dims=2)
+    n = q_out.shape[0]
+    vd = int(v_pages.shape[3])
+    width = (H + G) * hd + G * vd
+    ld = _cols(qkv, "qkv", width)
+    _need(q_weight, "q_weight", torch.float32, 1)
+    _need(k_weight, "k_weight", torch.float32, 1)
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != width:
+            raise KernelError("qk_row_norm_kv_write: bias must have one entry per projected column")
+    if tuple(q_out.shape) != (n, H * hd) or qkv.shape[0] != n or q_weight.shape[0] != H * hd or k_weight.shape[0] != G * hd:
+        raise KernelError("qk_row_norm_kv_write: qkv, q_out or a weight has the wrong shape")
+    _need(positions, "positions", torch.int32, 1)
+    _need(slot_of_token, "slot_of_token", torch.int32, 1)
+    _need(block_table, "block_table", torch.int32, 2)
+    _need(k_pages, "k_pages", q_out.dtype, 4)
+    _need(v_pages, "v_pages", q_out.dtype, 4)
+    if tuple(k_pages.shape[1:]) != (G, page_tokens, hd) or tuple(v_pages.shape[:3]) != tuple(k_pages.shape[:3]):
+        raise KernelError("cache pages must be [pages, G, page_tokens, head_dim] (values: their own width)")
+    lib = build.load("elementwise")
+    _check(lib.hk_qk_row_norm_kv_write(
+        _ptr(qkv), ctypes.c_longlong(ld), _ptr(bias), _ptr(q_out), _dt(q_out), _ptr(q_weight), _ptr(k_weight), ctypes.c_float(q_count),
+        ctypes.c_float(k_count), ctypes.c_float(eps), _ptr(positions), _ptr(slot_of_token), _ptr(block_table), int(block_table.shape[1]),
+        _ptr(k_pages), _ptr(v_pages), n, H, G, hd, vd, int(page_tokens), 1 if write_kv else 0, *_query_factor(q_factor), _stream()),
+        "qk_row_norm_kv_write")
 
 
 def maps_rope_kv_write(x, q_out, cos, sin, rotary_dim: int, positions, slot_of_token, block_table, k_pages, v_pages,
@@ -413,7 +513,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool =
 
 def paged_attention(q, k_pages, v_pages, block_table, positions, slot_of_token, out, n_heads, n_kv_heads,
                     head_dim, page_tokens, window: int, scale: float, plan=None, sink: bool = False, sinks=None,
-                    softcap: float = 0.0, chunk: int = 0, gate=None, gate_scale: float = 1.0) -> None:
+                    softcap: float = 0.0, chunk: int = 0, gate=None, gate_scale: float = 1.0, dist=None, dist_log2=None) -> None:
     """out[t, h, :] = softmax_j(scale * q[t, h] . k[j]) v[j] over the keys j in
     [max(0, p - window + 1), p] (all of [0, p] when window <= 0) of the token's request, read
     through its block-table row; p = positions[t].  `plan` carries the per-request tiling the
@@ -424,7 +524,8 @@ def paged_attention(q, k_pages, v_pages, block_table, positions, slot_of_token, 
     that float32 [H] tensor is given: p_j = exp(s_j) / (exp(sink) + sum exp(s_j)).
     `softcap` c > 0: scores become c * tanh(score / c).  `chunk` s > 0: a token sees no key before the start of its own
     block of s positions.  `gate` (a float32 column slice [n, H*vd] of a projection's output): the result is
-    multiplied by gate_scale * sigmoid(gate)."""
+    multiplied by gate_scale * sigmoid(gate).  `dist` float32 [H, N]: dist[h, min(n, N - 1)] is added to the (scaled, capped)
+    score of a key n positions back; `dist_log2`: the same table times log2(e), which the flash kernels read."""
     _need(q, "q", dims=2)
     _need(out, "out", q.dtype, 2)
     _need(k_pages, "k_pages", q.dtype, 4)
@@ -454,12 +555,18 @@ def paged_attention(q, k_pages, v_pages, block_table, positions, slot_of_token, 
         gate_ld = _cols(gate, "gate", H * vd)
         if gate.shape[0] != n:
             raise KernelError("paged_attention: one row of gate logits per token")
+    for name, t in (("dist", dist), ("dist_log2", dist_log2)):
+        if t is not None:
+            _need(t, name, torch.float32, 2)
+            if t.shape[0] != H or t.shape[1] < 1:
+                raise KernelError(f"paged_attention: {name} must be [heads, distances]")
     choice = _forced["attention"]
-    if q.dtype == torch.bfloat16 and choice != "generic" and plan is not None and v_pages is not None and vd == hd:
+    if q.dtype == torch.bfloat16 and choice != "generic" and plan is not None and v_pages is not None and vd == hd \
+            and (dist is None or dist_log2 is not None):
         from . import attention_fast
         done = attention_fast.run(q, k_pages, v_pages, block_table, out, H, G, hd, page_tokens, window, scale, plan,
                                   allow_tma=choice != "flash_cp", sink=sink, sinks=sinks, softcap=softcap, chunk=chunk,
-                                  gate=gate, gate_scale=gate_scale)
+                                  gate=gate, gate_scale=gate_scale, dist=dist_log2 if dist is not None else None)
         if done:
             if gate is not None and done != attention_fast.GATED:
                 sigmoid_gate(out, gate, out, gate_scale)
@@ -471,8 +578,8 @@ def paged_attention(q, k_pages, v_pages, block_table, positions, slot_of_token, 
         _ptr(q), _ptr(k_pages), _ptr(v_pages if v_pages is not None else k_pages), _dt(q), _ptr(block_table),
         int(block_table.shape[1]), _ptr(positions), _ptr(slot_of_token), _ptr(out), n, H, G, hd, int(page_tokens), int(window),
         ctypes.c_float(scale), vd, 1 if sink else 0, _ptr(sinks), ctypes.c_float(softcap), int(chunk),
-        vd if v_pages is not None else hd, _ptr(gate), ctypes.c_longlong(gate_ld), ctypes.c_float(gate_scale), _stream()),
-        "paged_attention")
+        vd if v_pages is not None else hd, _ptr(gate), ctypes.c_longlong(gate_ld), ctypes.c_float(gate_scale), _ptr(dist),
+        int(dist.shape[1]) if dist is not None else 0, _stream()), "paged_attention")
 
 
 def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
@@ -865,6 +972,43 @@ def state_space_scan(xbc, dt_logit, dt_bias, a_log, skip, segments, state, out, 
                                        N, dv, 1 if segments.shape[0] == n else 0, _stream()), "state_space_scan")
 
 
+def gla_decay(hid, w2, bias, tau: float, out) -> None:
+    """out[t, c] = log2(sigmoid(z)^(1 / tau)), z = sum_r w2[c, r] hid[t, r] + bias[c]: the log decays of a linear attention
+    with a decay per key channel.  hid a float32 column slice [n, R], w2 float32 [K, R], bias float32 [K], out float32 [n, K]."""
+    _need(w2, "w2", torch.float32, 2)
+    K, R = w2.shape
+    ldh = _cols(hid, "hid", R)
+    _need(bias, "bias", torch.float32, 1)
+    _need(out, "out", torch.float32, 2)
+    if tuple(out.shape) != (hid.shape[0], K) or bias.shape[0] != K or not tau > 0:
+        raise KernelError("gla_decay: shapes do not fit, or tau is not positive")
+    lib = build.load("gated_linear")
+    _check(lib.hk_gla_decay(_ptr(hid), ctypes.c_longlong(ldh), int(R), _ptr(w2), _ptr(bias), _ptr(out), out.shape[0], int(K),
+                            ctypes.c_float(tau), _stream()), "gla_decay")
+
+
+def gla_scan(q, k, v, la, segments, state, out, n_heads: int, key_dim: int, value_dim: int, q_scale: float) -> None:
+    """Linear attention with a decay per key channel over the rows of every segment, per head, S = state[slot, head] float32
+    (stored [dv, dk]):
+        S <- diag(2^la) S + k v^T;  out = S^T (q_scale q)
+    q, k [n, H*dk] and v [n, H*dv]: float32 column slices of ONE matrix; la float32 [n, H*dk]; out float32 [n, H*dv]."""
+    H, dk, dv = n_heads, key_dim, value_dim
+    ld = _cols(q, "q", H * dk)
+    if _cols(k, "k", H * dk) != ld or _cols(v, "v", H * dv) != ld:
+        raise KernelError("gla_scan: q, k and v must be slices of one matrix")
+    _need(la, "la", torch.float32, 2)
+    _need(segments, "segments", torch.int32, 2)
+    _need(state, "state", torch.float32, 4)
+    _need(out, "out", torch.float32, 2)
+    n = q.shape[0]
+    if tuple(state.shape[1:]) != (H, dv, dk) or tuple(out.shape) != (n, H * dv) or tuple(la.shape) != (n, H * dk) or segments.shape[1] != 3:
+        raise KernelError("gla_scan: shapes do not fit")
+    lib = build.load("gated_linear")
+    _check(lib.hk_gla_walk(_ptr(q), _ptr(k), _ptr(v), ctypes.c_longlong(ld), _ptr(la), _ptr(segments), int(segments.shape[0]),
+                           _ptr(state), _ptr(out), H, dk, dv, ctypes.c_float(q_scale), 1 if segments.shape[0] == n else 0, _stream()),
+           "gla_scan")
+
+
 def gated_part_norm(y, z, weight, eps: float, out, parts: int) -> None:
     """u = y * silu(z); out = every one of `parts` equal parts of a row of u over sqrt(mean(u^2) + eps) of that part, times
     weight.  y float32 [n, W], z a float32 column slice [n, W], weight float32 [W]."""
@@ -963,6 +1107,15 @@ def scaled_sum(out, a, alpha: float, b=None, beta: float = 0.0, accumulate: bool
                              ctypes.c_longlong(out.numel()), 1 if accumulate else 0, _stream()), "scaled_sum")
 
 
+def soft_cap(x: torch.Tensor, cap: float) -> None:
+    """x <- cap * tanh(x / cap) in place (float32)."""
+    _need(x, "x", torch.float32)
+    if not cap > 0:
+        raise KernelError("soft_cap: the cap must be positive")
+    lib = build.load("elementwise")
+    _check(lib.hk_soft_cap(_ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(cap), _stream()), "soft_cap")
+
+
 def narrow(x, out) -> None:
     """out = x (float32) rounded to out's type, element by element."""
     _need(x, "x", torch.float32)
@@ -1000,7 +1153,7 @@ ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_all": 2}
 
 
 def route_topk(x, w_router, ids, weights, scores: str = "softmax", correction=None, groups: int = 0, keep: int = 0,
-               scale: float = 1.0, norm_eps: float = 0.0, extra_out=None) -> None:
+               scale: float = 1.0, norm_eps: float = 0.0, extra_out=None, bias=None) -> None:
     """Per row of x [n, d]: the `top` = ids.shape[1] largest of the E float32 router logits x . w_router[e]
     (w_router float32 [E, d]; the lower index wins a tie), and the softmax over the chosen logits.
     scores 'sigmoid': every expert's score is s = sigmoid(logit); the choice is made on s + correction (float32 [E], or
@@ -1008,7 +1161,7 @@ def route_topk(x, w_router, ids, weights, scores: str = "softmax", correction=No
     sum of its two largest choice scores; the others count as minus infinity); weights = s / (sum of the chosen s +
     norm_eps) * scale.  `extra_out` float32 [n, X]: w_router has X more rows behind the experts', and the sigmoids of their
     logits are written there.  scores 'softmax_all': s = softmax over all E logits, the choice is made on s + correction,
-    weights = s * scale (not renormalised)."""
+    weights = s * scale (not renormalised).  `bias` (float32, one entry per row of w_router, or None) is added to the logits."""
     _need(x, "x", dims=2)
     _need(w_router, "w_router", torch.float32, 2)
     _need(ids, "ids", torch.int32, 2)
@@ -1027,10 +1180,14 @@ def route_topk(x, w_router, ids, weights, scores: str = "softmax", correction=No
         _need(correction, "correction", torch.float32, 1)
         if correction.shape[0] != E:
             raise KernelError("route_topk: one correction per expert")
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != E + extra:
+            raise KernelError("route_topk: one bias per row of the router")
     lib = build.load("routed")
     _check(lib.hk_route_topk(_ptr(x), _dt(x), _ptr(w_router), _ptr(ids), _ptr(weights), n, d, E, ids.shape[1],
                              ROUTE_SCORES[scores], _ptr(correction), int(groups), int(keep), ctypes.c_float(scale),
-                             ctypes.c_float(norm_eps), extra, _ptr(extra_out), _stream()), "route_topk")
+                             ctypes.c_float(norm_eps), extra, _ptr(extra_out), _ptr(bias), _stream()), "route_topk")
 
 
 def route_sort(ids, n_experts: int, offsets, perm, inv, tiles) -> None:

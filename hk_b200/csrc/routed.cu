@@ -4,7 +4,8 @@
 // on its number of rows alone (a decode step through it can be captured in a graph):
 //   1. route:   one block per token takes the E router logits (float32 products of the token's vector with
 //               the router's rows, summed in a fixed order), picks the `top` largest (the lower index wins a
-//               tie) and gives them the softmax over the chosen logits as weights.  A second mode scores every
+//               tie) and gives them the softmax over the chosen logits as weights (`bias`: a float per expert that is
+//               added to its logit first).  A second mode scores every
 //               expert by itself: s = sigmoid(logit); the choice is made on s + correction (a float per expert),
 //               optionally among the experts of the best `keep` of `groups` equal groups of neighbours (a
 //               group's score: the sum of its two largest choice scores), and the weights are the chosen
@@ -41,6 +42,7 @@ struct RouteOpts {
   float scale, norm_eps;     // mode 1: weights = s / (sum s + norm_eps) * scale; mode 2: weights = s * scale
   int extra;                 // rows of w behind the E experts' rows
   float* extra_out;          // [n, extra]: the sigmoids of those rows' logits
+  const float* bias;         // [E + extra]: added to the logits (null: nothing)
 };
 
 template <typename T>
@@ -91,7 +93,7 @@ route_topk_kernel(const T* __restrict__ x, const float* __restrict__ w, int* __r
     float sum = 0.f;
 #pragma unroll
     for (int wv = 0; wv < RK_WARPS; ++wv) sum += part[(size_t)wv * E + e];
-    z[e] = sum;
+    z[e] = opt.bias != nullptr ? sum + opt.bias[e] : sum;
   }
   __syncthreads();
   if (wid != 0) return;
@@ -204,13 +206,13 @@ route_topk_kernel(const T* __restrict__ x, const float* __restrict__ w, int* __r
 
 HK_API int hk_route_topk(const void* x, int dtype, const float* w, int* ids, float* weights, int n, int d, int E, int top, int mode,
                          const float* correction, int groups, int keep, float scale, float norm_eps, int extra, float* extra_out,
-                         void* stream) {
+                         const float* bias, void* stream) {
   if (n <= 0) return 0;
   if (E < 1 || top < 1 || top > E || top > 32 || E > 2048 || mode < 0 || mode > 2 || extra < 0 || extra > 64) return HK_ERR_UNSUPPORTED;
   if (mode == 0 && (correction != nullptr || groups != 0 || extra != 0)) return HK_ERR_UNSUPPORTED;
   if (mode == 2 && (groups != 0 || extra != 0)) return HK_ERR_UNSUPPORTED;
   if (groups < 0 || (groups > 0 && (E % groups || keep < 1 || keep > groups)) || (extra > 0 && extra_out == nullptr)) return HK_ERR_UNSUPPORTED;
-  const RouteOpts opt = {mode, correction, groups, keep, scale, norm_eps, extra, extra_out};
+  const RouteOpts opt = {mode, correction, groups, keep, scale, norm_eps, extra, extra_out, bias};
   const size_t smem = ((size_t)(RK_WARPS + 1) * (E + extra) + E + 2 * groups) * sizeof(float);
   dim3 grid((unsigned)n);
   cudaStream_t s = (cudaStream_t)stream;

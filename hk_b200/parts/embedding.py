@@ -4,7 +4,7 @@ Embedding: x[t, :] = E[token_t, :] widened to the float32 residual
 (src/engine/cpu_backend.zig:237-244), times `scale` (1 unless a design multiplies its embeddings).  Head: final norm on the wanted rows only, then
 logits = xb W_out^T in float32 (cpu_backend.zig:329-357); W_out is `lm_head.weight` when
 the file has it, else the embedding table when the configuration ties them
-(src/engine/weights.zig:124-129; src/convert/hf.zig:313,481-484)."""
+(src/engine/weights.zig:124-129; src/convert/hf.zig:313,481-484).  `softcap` c bounds the logits: z <- c tanh(z / c)."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -37,8 +37,9 @@ class TokenEmbedding(Part):
 class OutputHead(Part):
     graph_safe = True   # reads the batch from device tensors only
 
-    def __init__(self, hidden: int, vocab: int, norm, name: str, tied_to: Optional[str] = None):
+    def __init__(self, hidden: int, vocab: int, norm, name: str, tied_to: Optional[str] = None, softcap: float = 0.0):
         self.hidden, self.vocab, self.norm, self.name, self.tied_to = hidden, vocab, norm, name, tied_to
+        self.softcap = float(softcap)          # 0: none
         self.weight = None
 
     def children(self):
@@ -59,4 +60,6 @@ class OutputHead(Part):
         self.norm.forward(residual, xb, rows)
         logits = torch.empty((n_rows, self.vocab), dtype=torch.float32, device=residual.device)
         ops.gemm(xb, self.weight, logits)
+        if self.softcap:
+            ops.soft_cap(logits, self.softcap)
         return logits

@@ -135,6 +135,7 @@ class RoutedFeedForward(Part):
     `scores="softmax_all"` is a third router: s = softmax(z) over all of its outputs, the choice is made on s + correction,
     and the weights are the chosen s themselves (times `weight_scale`).  `identity`: the router has that many further
     outputs behind the experts' which stand for no feed-forward: such a choice gives back xb itself, times its weight.
+    `router_bias`: a tensor with one entry per router output that is added to the logits (for every kind of scores).
     `act`, `limit`, `slope` are the experts' gated activation (silu, or the clamped form of `SwiGLUFeedForward`);
     `out_scale` is a factor on the whole result."""
     graph_safe = True   # reads the batch from device tensors only; launches depend on the row count alone
@@ -145,7 +146,7 @@ class RoutedFeedForward(Part):
     def __init__(self, hidden: int, intermediate: int, n_experts: int, top: int, prefix: str, names=None,
                  scores: str = "softmax", correction: bool = False, groups: int = 0, keep: int = 0, weight_scale: float = 1.0,
                  norm_eps: float = 0.0, shared=None, shared_gated: bool = False, identity: int = 0, act: str = "silu",
-                 limit: float = 0.0, slope: float = 1.0, out_scale: float = 1.0):
+                 limit: float = 0.0, slope: float = 1.0, out_scale: float = 1.0, router_bias: bool = False):
         if identity < 0 or not 1 <= top <= n_experts + identity or top > 32:
             raise ValueError(f"top = {top} must be in 1..min(experts, 32) (experts = {n_experts}, identities = {identity})")
         if scores not in ops.ROUTE_SCORES:
@@ -158,6 +159,8 @@ class RoutedFeedForward(Part):
             raise ValueError("a correction, groups, a factor on the weights and a gated shared part belong to scores='sigmoid'")
         if groups and (n_experts % groups or not 1 <= keep <= groups):
             raise ValueError(f"{n_experts} experts do not form {groups} equal groups of which {keep} are kept")
+        if router_bias and shared_gated:
+            raise ValueError("the gate of a shared part is a row of the router's product and has no bias")
         if shared_gated and shared is None:
             raise ValueError("shared_gated needs a shared part")
         self.hidden, self.F, self.E, self.top, self.prefix = hidden, intermediate, n_experts, top, prefix
@@ -165,11 +168,11 @@ class RoutedFeedForward(Part):
         self.weight_scale, self.norm_eps = float(weight_scale), float(norm_eps)
         self.shared, self.shared_gated = shared, bool(shared_gated)
         self.identity, self.act, self.limit, self.slope = int(identity), act, float(limit), float(slope)
-        self.out_scale = float(out_scale)
-        self.names = {"router": "router", "expert": "e{}.", "gate": "gate", "up": "up", "down": "down",
+        self.out_scale, self.router_bias = float(out_scale), bool(router_bias)
+        self.names = {"router": "router", "router_bias": "router.b", "expert": "e{}.", "gate": "gate", "up": "up", "down": "down",
                       "correction": "correction", "shared_gate": "shared.sg"}
         self.names.update(names or {})
-        self.w_router = self.w_gate_up = self.w_down = self.w_correction = None
+        self.w_router = self.w_gate_up = self.w_down = self.w_correction = self.b_router = None
 
     def children(self):
         return (self.shared,) if self.shared is not None else ()
@@ -180,6 +183,8 @@ class RoutedFeedForward(Part):
     def own_param_specs(self) -> Dict[str, ParamSpec]:
         outputs = self.E + self.identity
         specs = {self.prefix + self.names["router"]: ParamSpec((outputs, self.hidden), MATRIX)}
+        if self.router_bias:
+            specs[self.prefix + self.names["router_bias"]] = ParamSpec((outputs,), VECTOR)
         if self.correction:
             specs[self.prefix + self.names["correction"]] = ParamSpec((outputs,), VECTOR)
         if self.shared_gated:
@@ -194,6 +199,8 @@ class RoutedFeedForward(Part):
         self.w_router = tensors[self.prefix + self.names["router"]].float().contiguous()    # the router runs in 32-bit
         if self.shared_gated:       # the shared part's gate is one more row of the router's product
             self.w_router = torch.cat([self.w_router, tensors[self.prefix + self.names["shared_gate"]].float()]).contiguous()
+        if self.router_bias:
+            self.b_router = tensors[self.prefix + self.names["router_bias"]]
         if self.correction:
             self.w_correction = tensors[self.prefix + self.names["correction"]]
         dt = precision.compute
@@ -237,7 +244,7 @@ class RoutedFeedForward(Part):
         weights = torch.empty((n, self.top), dtype=torch.float32, device=dev)
         shared_gate = torch.empty((n, 1), dtype=torch.float32, device=dev) if self.shared_gated else None
         ops.route_topk(xb, self.w_router, ids, weights, self.scores, self.w_correction, self.groups, self.keep, self.weight_scale,
-                       self.norm_eps, shared_gate)
+                       self.norm_eps, shared_gate, self.b_router)
         if RoutedFeedForward.route_log is not None:
             RoutedFeedForward.route_log.append(ids.clone())
         shared_y = None
