@@ -5,14 +5,14 @@ from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichNormBlock
 from .embedding import OutputHead, TokenEmbedding
 from .feed_forward import PolyNormFeedForward, RoutedFeedForward, SquaredReLUFeedForward, SwiGLUFeedForward
 from .latent_attention import LatentAttention
-from .norm import RMSNorm
+from .norm import LayerNorm, RMSNorm
 from .parallel import ParallelMixer
 from .position import RopeScaling, RotaryEmbedding
-from .recurrent import GatedDeltaRule, GeneralDeltaRule, MLSTM, MinGRU, Retention, ShortConvolution, StateSpace
+from .recurrent import GatedDeltaRule, GatedLinearAttention, GeneralDeltaRule, MLSTM, MinGRU, Retention, ShortConvolution, StateSpace
 from .side_input import TokenSideInput
 
 __all__ = [
-    "DifferentialAttention", "GQAAttention", "GatedDeltaRule", "Retention", "ShortConvolution", "GeneralDeltaRule", "MLSTM", "ParallelBlock", "ParallelMixer", "SquaredReLUFeedForward", "StateSpace", "TokenSideInput", "KVCacheSpec", "LatentAttention", "MinGRU", "PostNormBlock", "PolyNormFeedForward", "RoutedFeedForward", "SandwichNormBlock", "MATRIX", "OutputHead", "ParamSpec", "Part", "Precision", "PreNormBlock",
+    "DifferentialAttention", "GQAAttention", "GatedDeltaRule", "GatedLinearAttention", "LayerNorm", "Retention", "ShortConvolution", "GeneralDeltaRule", "MLSTM", "ParallelBlock", "ParallelMixer", "SquaredReLUFeedForward", "StateSpace", "TokenSideInput", "KVCacheSpec", "LatentAttention", "MinGRU", "PostNormBlock", "PolyNormFeedForward", "RoutedFeedForward", "SandwichNormBlock", "MATRIX", "OutputHead", "ParamSpec", "Part", "Precision", "PreNormBlock",
     "RMSNorm", "RopeScaling", "RotaryEmbedding", "StateSpec", "StepTables", "SwiGLUFeedForward", "TABLE", "TokenEmbedding", "VECTOR",
     "part_class", "register_part",
 ]

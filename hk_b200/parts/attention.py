@@ -30,17 +30,25 @@ Further parameters, for designs other than the reference's:
   `gate` multiplies the concatenated heads' outputs, before W_o, element by element with sigmoid(W_g x) of the
   mixer's own input (tensor `g` [H * v_head_dim, hidden], fused into the q/k/v product); `out_scale` is a factor on
   the mixer's result that the gate carries;
-  `names` renames the tensors (keys q, k, v, o, q_norm, k_norm, sink, gate, and q_bias, k_bias, v_bias, o_bias).
+  `qk_norm_rows` norms q (and k) over all of its rows at once, before they are split into heads, with weights of that size
+  (tensors `q_norm` [H * head_dim], `k_norm` [G * head_dim]), instead of head by head;
+  `q_factor` (coef, every) multiplies a query at position p by 1 + coef ln(floor((p + 1) / every) + 1);
+  `bias_max` D adds a learned number per head and distance to the scaled scores (tensor `rel` [B, H]): with n the distance
+  of a key, row n of the table for n < B/2, else row min(B - 1, B/2 + floor(ln(n / (B/2)) / ln(D / (B/2)) (B - B/2)));
+  `pad_to` fills the heads of q, k and v up with zeros to that width in the cache and in the kernels (`padded_head`), where
+  the sizes themselves are none that the tensor-core kernels take: a zero changes no score and no value;
+  `names` renames the tensors (keys q, k, v, o, q_norm, k_norm, sink, gate, rel, and q_bias, k_bias, v_bias, o_bias).
 """
 from __future__ import annotations
 
 import math
+from fractions import Fraction
 from typing import Dict, Optional
 
 import torch
 
 from ..csrc import ops
-from .base import KVCacheSpec, MATRIX, VECTOR, ParamSpec, Part, Precision, StepTables, register_part
+from .base import KVCacheSpec, MATRIX, VECTOR, ParamSpec, Part, Precision, StepTables, register_part, stacked_rows
 from .position import RotaryEmbedding
 
 
@@ -82,8 +90,63 @@ def flash_plan(ctx, key):
     return attention_fast.plan_on_device(info, arrays["items"], arrays.get("merge"))
 
 
+def distance_starts(buckets: int, furthest) -> list:
+    """The first distance that each row >= B/2 of a distance table of `buckets` rows serves, row B/2 first, by exact
+    arithmetic: row B/2 + k starts at the least n with (n / half)^m >= (furthest / half)^k, half = B/2, m = B - half."""
+    half = buckets // 2
+    m = buckets - half
+    if buckets < 2:
+        return []
+    if not furthest > half:
+        raise ValueError(f"a distance bias of {buckets} rows must reach further than {half} positions, not {furthest}")
+    ratio = Fraction(furthest) / half
+    starts = []
+    for k in range(m):
+        n = max(half, int(half * float(ratio) ** (k / m)) - 2)
+        while Fraction(n, half) ** m < ratio ** k:
+            n += 1
+        starts.append(n)
+    return starts
+
+
+def distance_table(rel: torch.Tensor, furthest) -> torch.Tensor:
+    """A bias by bucket of distance, rel [B, H], as one number per head and distance, [H, N]: entry N - 1 serves every
+    distance from N - 1 on."""
+    B = int(rel.shape[0])
+    if B < 2:
+        rows = [0]
+    else:
+        half, starts = B // 2, distance_starts(B, furthest)
+        rows = list(range(half))
+        for k, start in enumerate(starts):
+            stop = starts[k + 1] if k + 1 < len(starts) else start + 1
+            rows += [half + k] * (stop - start)
+    return rel.float()[torch.tensor(rows, device=rel.device)].t().contiguous()
+
+
+def padded_head(head_dim: int, v_head_dim: int) -> Optional[int]:
+    """The width to which heads of these sizes are filled up for the tensor-core kernels, or None where they are taken as
+    they are (or where no kernel takes them)."""
+    from ..csrc import attention_fast
+    if head_dim == v_head_dim and attention_fast.supported(head_dim, 1):
+        return None
+    widest = max(head_dim, v_head_dim)
+    return 64 if widest <= 64 else 128 if widest <= 128 else None
+
+
+def _filled(t: torch.Tensor, heads: int, width: int) -> torch.Tensor:
+    """The rows [heads * w, ...] with every head's w rows filled up with zeros to `width`."""
+    w = t.shape[0] // heads
+    if w == width:
+        return t
+    out = torch.zeros((heads, width) + tuple(t.shape[1:]), dtype=t.dtype, device=t.device)
+    out[:, :w] = t.reshape((heads, w) + tuple(t.shape[1:]))
+    return out.reshape((heads * width,) + tuple(t.shape[1:]))
+
+
 class GQAAttention(Part):
     graph_safe = True   # reads the batch from device tensors only
+    takes_projection = True     # `forward` can be handed the product with `in_weight` (`proj`)
 
     def __init__(self, hidden: int, n_heads: int, n_kv_heads: int, head_dim: int, prefix: str,
                  qk_norm_eps: Optional[float] = None, position: Optional[RotaryEmbedding] = None,
@@ -91,19 +154,33 @@ class GQAAttention(Part):
                  o_bias: bool = False, qk_norm_after: bool = False, qk_norm_weight: bool = True,
                  value_from_key: bool = False, v_head_dim: Optional[int] = None, sink: bool = False,
                  names: Optional[Dict[str, str]] = None, sink_weights: bool = False, softcap: Optional[float] = None,
-                 chunk: Optional[int] = None, gate: bool = False, out_scale: float = 1.0):
+                 chunk: Optional[int] = None, gate: bool = False, out_scale: float = 1.0, qk_norm_rows: bool = False, q_factor=None,
+                 bias_max=None, bias_rows: Optional[int] = None, pad_to: Optional[int] = None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} heads are not a multiple of {n_kv_heads} key/value heads")
         if head_dim > 256 or head_dim < 2:
             raise ValueError(f"head_dim {head_dim} is outside 2..256")
         if position is not None and position.rotary_dim > head_dim:
             raise ValueError("the rotary width exceeds head_dim")
-        self.hidden, self.H, self.G, self.hd = hidden, n_heads, n_kv_heads, head_dim
-        self.vd = head_dim if v_head_dim is None else int(v_head_dim)
+        # dim and vdim are the model's sizes, hd and vd those of the cache and the kernels
+        self.hidden, self.H, self.G, self.hd, self.dim = hidden, n_heads, n_kv_heads, head_dim, head_dim
+        self.vd = self.vdim = head_dim if v_head_dim is None else int(v_head_dim)
         if not 1 <= self.vd <= 256 or (self.vd > head_dim and value_from_key):
             raise ValueError(f"value size {self.vd} must be in 1..256, and at most head_dim when the values are the keys")
         if sink_weights and not sink:
             raise ValueError("sink_weights needs sink")
+        self.qk_norm_rows = bool(qk_norm_rows)
+        if qk_norm_rows and (qk_norm_eps is None or not qk_norm_weight or qk_norm_after or value_from_key or position is not None):
+            raise ValueError("a norm over the whole projection has weights, an eps and neither a rotation nor tied values")
+        if q_factor is not None and int(q_factor[1]) < 1:
+            raise ValueError("the queries' factor needs a positive number of positions per step")
+        self.q_factor = (float(q_factor[0]), int(q_factor[1])) if q_factor is not None else None
+        self.bias_max, self.bias_rows = bias_max, bias_rows
+        self.dist = self.dist_log2 = None
+        if pad_to is not None:
+            if pad_to < max(head_dim, self.vd) or value_from_key or (qk_norm_eps is not None and not qk_norm_rows):
+                raise ValueError("heads can be filled up to a larger width, with values of their own and no norm per head")
+            self.hd = self.vd = int(pad_to)
         self.sink_weights, self.gate = bool(sink_weights), bool(gate)
         if out_scale != 1.0 and not gate:
             raise ValueError("out_scale rides on the output gate: it needs gate=True")
@@ -115,7 +192,7 @@ class GQAAttention(Part):
         self.qk_norm_after, self.qk_norm_weight = bool(qk_norm_after), bool(qk_norm_weight)
         self.value_from_key, self.sink = bool(value_from_key), bool(sink)
         self.names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
-                      "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sink", "gate": "g_proj.weight",
+                      "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sink", "gate": "g_proj.weight", "rel": "rel",
                       "q_bias": "q_proj.bias",
                       "k_bias": "k_proj.bias", "v_bias": "v_proj.bias", "o_bias": "o_proj.bias"}
         self.names.update(names or {})
@@ -149,26 +226,29 @@ class GQAAttention(Part):
         return (self.position,) if self.position is not None else ()
 
     def own_param_specs(self) -> Dict[str, ParamSpec]:
-        p, H, G, hd, d, nm = self.prefix, self.H, self.G, self.hd, self.hidden, self.names
+        p, H, G, hd, vd, d, nm = self.prefix, self.H, self.G, self.dim, self.vdim, self.hidden, self.names
         specs = {
             p + nm["q"]: ParamSpec((H * hd, d), MATRIX),
             p + nm["k"]: ParamSpec((G * hd, d), MATRIX),
-            p + nm["o"]: ParamSpec((d, H * self.vd), MATRIX),
+            p + nm["o"]: ParamSpec((d, H * vd), MATRIX),
         }
         if not self.value_from_key:
-            specs[p + nm["v"]] = ParamSpec((G * self.vd, d), MATRIX)
+            specs[p + nm["v"]] = ParamSpec((G * vd, d), MATRIX)
         if self.sink_weights:
             specs[p + nm["sink"]] = ParamSpec((H,), VECTOR)
         if self.gate:
-            specs[p + nm["gate"]] = ParamSpec((H * self.vd, d), MATRIX)
+            specs[p + nm["gate"]] = ParamSpec((H * vd, d), MATRIX)
+        if self.bias_max is not None:
+            specs[p + nm["rel"]] = ParamSpec((self.bias_rows or -1, H), VECTOR)      # -1: as many rows as the file's tensor has
         if self.qk_norm_eps is not None and self.qk_norm_weight:
-            specs[p + nm["q_norm"]] = ParamSpec((hd,), VECTOR, "one_plus_normal")
-            specs[p + nm["k_norm"]] = ParamSpec((hd,), VECTOR, "one_plus_normal")
+            q_rows, k_rows = (H * hd, G * hd) if self.qk_norm_rows else (hd, hd)
+            specs[p + nm["q_norm"]] = ParamSpec((q_rows,), VECTOR, "one_plus_normal")
+            specs[p + nm["k_norm"]] = ParamSpec((k_rows,), VECTOR, "one_plus_normal")
         if self.qkv_bias:
             specs[p + nm["q_bias"]] = ParamSpec((H * hd,), VECTOR)
             specs[p + nm["k_bias"]] = ParamSpec((G * hd,), VECTOR)
             if not self.value_from_key:
-                specs[p + nm["v_bias"]] = ParamSpec((G * self.vd,), VECTOR)
+                specs[p + nm["v_bias"]] = ParamSpec((G * vd,), VECTOR)
         if self.o_bias:
             specs[p + nm["o_bias"]] = ParamSpec((d,), VECTOR)
         return specs
@@ -179,22 +259,29 @@ class GQAAttention(Part):
     def own_bind(self, tensors, precision: Precision) -> None:
         p, nm = self.prefix, self.names
         parts = "qk" if self.value_from_key else "qkv"
-        qkv = [tensors[p + nm[c]] for c in parts]
+        heads = {"q": (self.H, self.hd), "k": (self.G, self.hd), "v": (self.G, self.vd)}
+        qkv = [_filled(tensors[p + nm[c]], *heads[c]) for c in parts]
         self._qkv_width = sum(int(t.shape[0]) for t in qkv)
         if self.gate:                        # the gate's logits are further columns of the same product
-            qkv.append(tensors[p + nm["gate"]])
+            qkv.append(_filled(tensors[p + nm["gate"]], self.H, self.vd))
         if self.sink_weights:
             self.sinks = tensors[p + nm["sink"]]
-        wide = torch.float32 if any(t.dtype == torch.float32 for t in qkv) else qkv[0].dtype    # one kept in 32-bit: all are
-        self.w_qkv = torch.cat([t.to(wide) for t in qkv], dim=0).contiguous()
+        self.w_qkv = stacked_rows(qkv)
         self.w_o = tensors[p + nm["o"]]
+        if self.vd != self.vdim:
+            self.w_o = _filled(self.w_o.t(), self.H, self.vd).t().contiguous()
         if self.qkv_bias:
-            self.b_qkv = torch.cat([tensors[p + nm[c + "_bias"]] for c in parts]).contiguous()
+            self.b_qkv = torch.cat([_filled(tensors[p + nm[c + "_bias"]], *heads[c]) for c in parts]).contiguous()
+        if self.bias_max is not None:
+            self.dist = distance_table(tensors[p + nm["rel"]], self.bias_max)
+            self.dist_log2 = (self.dist * math.log2(math.e)).contiguous()
         if self.o_bias:
             self.b_o = tensors[p + nm["o_bias"]]
         if self.qk_norm_eps is not None and self.qk_norm_weight:
             self.q_norm = tensors[p + nm["q_norm"]]
             self.k_norm = tensors[p + nm["k_norm"]]
+            if self.qk_norm_rows:
+                self.q_norm, self.k_norm = _filled(self.q_norm, self.H, self.hd), _filled(self.k_norm, self.G, self.hd)
         from ..csrc import attention_fast
         if precision.compute == torch.bfloat16 and self._flash_takes():
             self._tables_key = ("paged_attention_items", self.window or 0, self.H, self.G, self.hd, self.sink, self.chunk, bool(self.softcap))
@@ -212,18 +299,29 @@ class GQAAttention(Part):
     def _plan(self, ctx):
         return flash_plan(ctx, self._tables_key)
 
+    @property
+    def in_weight(self) -> torch.Tensor:
+        """What the mixer's input is multiplied with first: q, k, v (and the gate) as one matrix."""
+        return self.w_qkv
+
+    @in_weight.setter
+    def in_weight(self, weight: torch.Tensor) -> None:
+        self.w_qkv = weight
+
     # -- one step ------------------------------------------------------------------------
     def forward(self, xb: torch.Tensor, residual: torch.Tensor, ctx, cache, write_cache: bool = True,
-                accumulate: bool = True) -> None:
+                accumulate: bool = True, proj=None, add_bias: bool = True) -> None:
         """`accumulate=False` stores the mixer's result in `residual` instead of adding it (a block that norms the
-        result before the residual sum)."""
+        result before the residual sum).  `proj`: the float32 product of xb with `in_weight`, where a pair of mixers has
+        made it along with its own; `add_bias=False` leaves the output projection's bias (`b_o`) to the caller."""
         n = xb.shape[0]
         H, G, hd = self.H, self.G, self.hd
         plan = self._plan(ctx) if xb.dtype == torch.bfloat16 else None
-        proj = torch.empty((n, self.w_qkv.shape[0]), dtype=torch.float32, device=xb.device)
-        ops.gemm(xb, self.w_qkv, proj)
-        qkv = proj[:, :self._qkv_width] if self.gate else proj
-        gate = proj[:, self._qkv_width:] if self.gate else None
+        if proj is None:
+            proj = torch.empty((n, self.w_qkv.shape[0]), dtype=torch.float32, device=xb.device)
+            ops.gemm(xb, self.w_qkv, proj)
+        qkv = proj[:, :self._qkv_width]
+        gate = proj[:, self._qkv_width:self._qkv_width + H * self.vd] if self.gate else None
         q = torch.empty((n, H * hd), dtype=xb.dtype, device=xb.device)
         cos = sin = None
         rot = 0
@@ -232,17 +330,23 @@ class GQAAttention(Part):
             cos, sin, rot = self.position.tables()
             pairing = getattr(self.position, "pairing", "half")
         # the projections' bias rides on the fused kernel's load
-        ops.qk_norm_rope_kv_write(
-            qkv, q, self.q_norm, self.k_norm, self.qk_norm_eps or 0.0, cos, sin, rot, ctx.positions,
-            ctx.slot_of_token, cache.block_table, cache.k_pages, cache.v_pages, H, G, hd, cache.page_tokens,
-            write_kv=write_cache, bias=self.b_qkv, pairing=pairing, norm_after=self.qk_norm_after,
-            tied_v=self.value_from_key)
+        if self.qk_norm_rows:
+            ops.qk_row_norm_kv_write(
+                qkv, q, self.q_norm, self.k_norm, H * self.dim, G * self.dim, self.qk_norm_eps, ctx.positions, ctx.slot_of_token,
+                cache.block_table, cache.k_pages, cache.v_pages, H, G, hd, cache.page_tokens, write_kv=write_cache, bias=self.b_qkv,
+                q_factor=self.q_factor)
+        else:
+            ops.qk_norm_rope_kv_write(
+                qkv, q, self.q_norm, self.k_norm, self.qk_norm_eps or 0.0, cos, sin, rot, ctx.positions,
+                ctx.slot_of_token, cache.block_table, cache.k_pages, cache.v_pages, H, G, hd, cache.page_tokens,
+                write_kv=write_cache, bias=self.b_qkv, pairing=pairing, norm_after=self.qk_norm_after,
+                tied_v=self.value_from_key, q_factor=self.q_factor)
         att = torch.empty((n, H * self.vd), dtype=xb.dtype, device=xb.device)
         ops.paged_attention(q, cache.k_pages, cache.v_pages, cache.block_table, ctx.positions, ctx.slot_of_token,
                             att, H, G, hd, cache.page_tokens, self.window or 0, self.scale,
                             plan=plan, sink=self.sink, sinks=self.sinks, softcap=self.softcap, chunk=self.chunk, gate=gate,
-                            gate_scale=self.out_scale)
-        ops.gemm(att, self.w_o, residual, accumulate=accumulate, bias=self.b_o)
+                            gate_scale=self.out_scale, dist=self.dist, dist_log2=self.dist_log2)
+        ops.gemm(att, self.w_o, residual, accumulate=accumulate, bias=self.b_o if add_bias else None)
 
 
 register_part("mixer", "gqa_attention", GQAAttention)

@@ -32,9 +32,13 @@ class PreNormBlock(Part):
     def forward(self, residual: torch.Tensor, ctx, caches, write_cache: bool = True) -> None:
         xb = torch.empty(residual.shape, dtype=ctx.precision.compute, device=residual.device)
         self.mixer_norm.forward(residual, xb)
-        self.mixer.forward(xb, residual, ctx, mixer_caches(self.mixer, caches), write_cache)
+        # a mixer that ends in a pass over the residual rows writes the feed-forward's input along with them
+        ahead = self.feed_forward is not None and hasattr(self.mixer, "takes_next_norm") and self.mixer.takes_next_norm(self.ffn_norm)
+        more = {"next_norm": self.ffn_norm, "next_out": xb} if ahead else {}
+        self.mixer.forward(xb, residual, ctx, mixer_caches(self.mixer, caches), write_cache, **more)
         if self.feed_forward is not None:
-            self.ffn_norm.forward(residual, xb)
+            if not ahead:
+                self.ffn_norm.forward(residual, xb)
             self.feed_forward.forward(xb, residual, ctx)
         if self.after is not None:
             self.after.forward(residual, ctx)

@@ -49,6 +49,12 @@ h // (n_heads / n_groups)):
       dt <- softplus(dt + dt_bias);   S <- exp(-exp(A_log) dt) S + dt B x^T;   o = S^T C + D x
       y = W_o (N(o * silu(z)) * norm_weight),   N over each of `norm_groups` equal parts of the n_heads * value_dim numbers
 
+`GatedLinearAttention` (per head a matrix state S [key_dim, value_dim], zero at the start; a decay per key channel):
+      q = W_q h * key_dim^(-1/2),  k = W_k h,  v = W_v h;   z = W_a2 (W_a1 h) + b;   alpha = sigmoid(z)^(1 / tau)
+      S <- diag(alpha) S + k v^T;   o = S^T q
+      y = W_o ((o / rms(o) per head) * norm_weight[value_dim] * silu(W_g h))
+  The width of W_a1 is read from the configuration or, at binding, from the tensor; W_a2 and everything behind it is float32.
+
 `ShortConvolution` is the causal convolution over a request's last `taps` rows per channel as a part of its own (tensors
 [channels, taps] by group of channels, an optional bias and silu, the request's last taps - 1 inputs as its state), for mixers
 other than the gated delta rule that put one behind their projections.
@@ -436,6 +442,66 @@ class StateSpace(_SegmentScan):
         ops.gemm(og, self.w_o, residual, accumulate=accumulate)
 
 
+class GatedLinearAttention(_SegmentScan):
+    kernel_libraries = ("gated_linear", "recurrent")
+    takes_projection = True     # `forward` can be handed the product with `in_weight` (`proj`)
+
+    def __init__(self, hidden: int, n_heads: int, key_dim: int, value_dim: int, tau: float, prefix: str, norm_eps: float,
+                 decay_rank: Optional[int] = None, q_scale: Optional[float] = None, names: Optional[Dict[str, str]] = None):
+        if not tau > 0:
+            raise ValueError("tau must be positive")
+        self.hidden, self.H, self.dk, self.dv = hidden, n_heads, key_dim, value_dim
+        self.tau, self.prefix, self.norm_eps = float(tau), prefix, float(norm_eps)
+        self.decay_rank = decay_rank         # None: whatever the file's tensor has (known at binding)
+        self.q_scale = float(q_scale) if q_scale is not None else key_dim ** -0.5
+        self.names = {"q": "q", "k": "k", "v": "v", "g": "g", "a1": "a1", "a2": "a2", "a_bias": "a2.b", "norm": "norm", "o": "o"}
+        self.names.update(names or {})
+        self.in_weight = self.w_o = self.w_a2 = self.a_bias = self.norm_weight = None
+        self.rank = 0
+
+    def own_param_specs(self) -> Dict[str, ParamSpec]:
+        p, nm, d = self.prefix, self.names, self.hidden
+        K, V = self.H * self.dk, self.H * self.dv
+        R = self.decay_rank if self.decay_rank is not None else -1      # -1: any size along that axis
+        return {
+            p + nm["q"]: ParamSpec((K, d), MATRIX), p + nm["k"]: ParamSpec((K, d), MATRIX),
+            p + nm["v"]: ParamSpec((V, d), MATRIX), p + nm["g"]: ParamSpec((V, d), MATRIX),
+            p + nm["a1"]: ParamSpec((R, d), MATRIX), p + nm["a2"]: ParamSpec((K, R), VECTOR), p + nm["a_bias"]: ParamSpec((K,), VECTOR),
+            p + nm["norm"]: ParamSpec((self.dv,), VECTOR, "one_plus_normal"), p + nm["o"]: ParamSpec((d, V), MATRIX),
+        }
+
+    def cache_spec(self):
+        return StateSpec((self.H, self.dv, self.dk), torch.float32)
+
+    def own_bind(self, tensors, precision: Precision) -> None:
+        p, nm = self.prefix, self.names
+        # one product gives q, k, v, the output gate's logits and the hidden layer of the decay's low-rank projection
+        self.in_weight = stacked_rows([tensors[p + nm[c]] for c in ("q", "k", "v", "g", "a1")])
+        self.rank = int(tensors[p + nm["a1"]].shape[0])
+        self.w_a2, self.a_bias = tensors[p + nm["a2"]], tensors[p + nm["a_bias"]]
+        if int(self.w_a2.shape[1]) != self.rank:
+            raise ValueError(f"'{p + nm['a2']}' takes {int(self.w_a2.shape[1])} inputs, '{p + nm['a1']}' gives {self.rank}")
+        self.w_o, self.norm_weight = tensors[p + nm["o"]], tensors[p + nm["norm"]]
+
+    def forward(self, xb: torch.Tensor, residual: torch.Tensor, ctx, cache, write_cache: bool = True,
+                accumulate: bool = True, proj=None) -> None:
+        """`proj`: the float32 product of xb with `in_weight`, where a pair of mixers has made it along with its own."""
+        n, dev = xb.shape[0], xb.device
+        K, V, H = self.H * self.dk, self.H * self.dv, self.H
+        if proj is None:
+            proj = torch.empty((n, self.in_weight.shape[0]), dtype=torch.float32, device=dev)
+            ops.gemm(xb, self.in_weight, proj)
+        a0 = 2 * K + 2 * V
+        la = torch.empty((n, K), dtype=torch.float32, device=dev)
+        ops.gla_decay(proj[:, a0:a0 + self.rank], self.w_a2, self.a_bias, self.tau, la)
+        o = torch.empty((n, V), dtype=torch.float32, device=dev)
+        ops.gla_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], la, self._segments(ctx), cache.state, o, H, self.dk,
+                     self.dv, self.q_scale)
+        og = torch.empty((n, V), dtype=xb.dtype, device=dev)
+        ops.head_out_gate(o, proj[:, 2 * K + V:a0], self.norm_weight, self.norm_eps, og, H, self.dv, act="silu")
+        ops.gemm(og, self.w_o, residual, accumulate=accumulate)
+
+
 class MLSTM(_SegmentScan):
     def __init__(self, hidden: int, n_heads: int, key_dim: int, value_dim: int, gate_cap: float, prefix: str, norm_eps: float,
                  den_eps: float = 1e-6, q_scale: Optional[float] = None, names: Optional[Dict[str, str]] = None):
@@ -493,6 +559,7 @@ class MLSTM(_SegmentScan):
 register_part("mixer", "general_delta_rule", GeneralDeltaRule)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
 register_part("mixer", "mlstm", MLSTM)
+register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "mingru", MinGRU)
 register_part("mixer", "retention", Retention)
 register_part("mixer", "state_space", StateSpace)
