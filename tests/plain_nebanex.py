@@ -49,6 +49,8 @@ def bucket(n, buckets, furthest):
     spaced evenly in ln(n) up to `furthest`, from where on the last row serves.  (A distance that falls on a boundary
     exactly belongs to the upper row; the 1e-9 keeps a logarithm's last bit from deciding that.)"""
     half = buckets // 2
+    if buckets < 2:
+        return 0
     if n < half:
         return n
     steps = math.log(n / half) / math.log(furthest / half) * (buckets - half)
