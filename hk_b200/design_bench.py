@@ -970,11 +970,165 @@ def gezavik_kernel_points(width: int, n: int, decode: bool, peaks: dict) -> dict
     return out
 
 
+def nebanex_shape(width: int, groups: int = 2, vocab: int = 32000) -> dict:
+    """Layer sizes that resemble a real model's: in every layer an attention with heads of 128, four query heads per key head,
+    32 rows of distance bias up to 1,024 positions, beside a gated linear attention whose heads keep states of 64 x 128; eight
+    experts of half the width of which two are used, and a shared expert."""
+    heads = width // 128
+    lhs = {"bias_max": 1024, "bias_rows": 32, "dim": 128, "heads": heads, "kv_heads": max(1, heads // 4), "scale": 1.0 / math.sqrt(128.0),
+           "vdim": 128, "q_temp": {"coef": 0.3, "every": 1024}}
+    rhs = {"decay_rank": 16, "dim": 64, "heads": heads, "tau": 16.0, "vdim": 128}
+    moe = {"kind": "moe", "expert": {"ff": width // 2}, "router": {"experts": 8, "top": 2}, "shared": {"ff": width // 2}}
+    layer = {"type": "parallel", "mixer": {"left": lhs, "right": rhs}, "mlp": moe}
+    return {"architecture": "Nebanex", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "logit_softcap": 30.0, "layers": [layer] * (4 * groups), "initializer_range": 0.02}
+
+
+def nebanex_kernel_points(width: int, n: int, decode: bool, peaks: dict) -> dict:
+    """The design's kernels alone at a layer of this width, each beside the like kernel of the Mifolorn (or Zazulix) decoder: one
+    request of n prompt tokens, or (decode) n requests that each bring one token (the attention over 2,047 cached ones; these
+    are timed as replays of a captured graph)."""
+    import numpy as np
+    import torch
+
+    from .csrc import attention_fast, ops
+    from .parts.attention import distance_table
+    dev = "cuda"
+    bw, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    out = {}
+
+    def note(name, us, nbytes, flops, peak_flops, like=None):
+        floor = max(nbytes / bw, flops / peak_flops if peak_flops else 0.0) * 1e6
+        out[name] = {"us": round(us, 1), "bytes": int(nbytes), "flops": int(flops), "roofline_us": round(floor, 2),
+                     "of_roofline": round(floor / us, 3), **({"like": like} if like else {})}
+
+    count, rows = (n, 1) if decode else (1, n)
+    _time_kernel = lambda fn: globals()["_time_kernel"](fn, replay=decode)      # decode steps replay a captured graph
+    sg = torch.tensor([[i, i * rows, rows] for i in range(count)], dtype=torch.int32, device=dev)
+    fp32 = FP32_TFLOPS * 1e12
+    bf = torch.bfloat16
+
+    # ---- gated linear attention: decays, recurrence, the output's norm and gate; the like scans at as many state entries
+    H, dk, dv, R = width // 128, 64, 128, 16
+    K, V = H * dk, H * dv
+    proj = torch.randn(n, 2 * K + 2 * V + R, device=dev) * 0.5
+    w2 = torch.randn(K, R, device=dev) * 0.3
+    ab = torch.full((K,), 2.0, device=dev)
+    la = torch.empty(n, K, device=dev)
+    us = _time_kernel(lambda: ops.gla_decay(proj[:, 2 * K + 2 * V:], w2, ab, 16.0, la))
+    note("gla_decay (low-rank logits to log decays)", us, n * (R + K) * 4 + K * (R + 1) * 4, 2.0 * n * K * R, fp32, like="rms_norm")
+    state = torch.zeros(count, H, dv, dk, device=dev)
+    o = torch.empty(n, V, device=dev)
+    us = _time_kernel(lambda: ops.gla_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], la, sg, state, o, H, dk, dv, dk ** -0.5))
+    note("gla_scan", us, 4 * (n * (3 * K + 2 * V) + 2 * count * H * dk * dv), 5.0 * n * H * dk * dv, fp32, like="gated_delta_scan (Mifolorn)")
+    Hd, Gd = width // 64, width // 128
+    Kd, Vd = Gd * 64, Hd * 64
+    act = torch.randn(n, 2 * Kd + Vd, device=dev) * 0.5
+    lg = torch.randn(n, 2 * Hd, device=dev)
+    zh = torch.zeros(Hd, device=dev)
+    st = torch.zeros(count, Hd, 64, 64, device=dev)
+    od = torch.empty(n, Vd, device=dev)
+    us = _time_kernel(lambda: ops.gated_delta_scan(act[:, :Kd], act[:, Kd:2 * Kd], act[:, 2 * Kd:], lg[:, :Hd], lg[:, Hd:], zh, zh, sg, st, od, Hd,
+                                                   Gd, 64, 64, 0.125, 1e-6))
+    note("gated_delta_scan (Mifolorn)", us, 4 * (n * (2 * Kd + 2 * Vd + 2 * Hd) + 2 * count * Hd * 64 * 64), 8.0 * n * Hd * 64 * 64, fp32)
+    projr = torch.randn(n, 3 * Hd * 64, device=dev) * 0.5
+    dec = torch.full((Hd,), 0.99, device=dev)
+    zero_pos = torch.zeros(n, dtype=torch.int32, device=dev)
+    W = Hd * 64
+    us = _time_kernel(lambda: ops.retention_scan(projr[:, :W], projr[:, W:2 * W], projr[:, 2 * W:], None, None, 0, zero_pos, dec, sg, st, od, Hd, 64,
+                                                 64, 0.125))
+    note("retention_scan (Zazulix)", us, 4 * (4 * n * W + 2 * count * Hd * 64 * 64), 4.0 * n * Hd * 64 * 64, fp32)
+    og = torch.empty(n, V, dtype=bf, device=dev)
+    wn = torch.ones(dv, device=dev)
+    us = _time_kernel(lambda: ops.head_out_gate(o, proj[:, 2 * K + V:2 * K + 2 * V], wn, 1e-6, og, H, dv, act="silu"))
+    note("head_out_gate (values of 128, shared weight, silu)", us, n * V * (4 + 4 + 2), 0, 0, like="head_out_gate (Mifolorn: values of 64)")
+    us = _time_kernel(lambda: ops.head_out_gate(o, proj[:, 2 * K + V:2 * K + 2 * V], wn[:64].contiguous(), 1e-6, og, 2 * H, dv // 2, act="silu"))
+    note("head_out_gate (Mifolorn: values of 64)", us, n * V * (4 + 4 + 2), 0, 0)
+
+    # ---- attention with a bias by distance and an output gate; Mifolorn's with its soft cap
+    Ha, Ga, hd, pt, context = width // 128, max(1, width // 512), 128, 64, 2047
+    sm = torch.cuda.get_device_properties(0).multi_processor_count
+    per = (context + 1) if decode else n
+    ppr = -(-per // pt)
+    table = torch.arange(count * ppr, dtype=torch.int32, device=dev).view(count, ppr).contiguous()
+    slots = list(range(count))
+    q_starts, q_lens = (list(range(n)), [1] * n) if decode else ([0], [n])
+    starts = [context] * n if decode else [0]
+    positions = torch.tensor([context] * n if decode else list(range(n)), dtype=torch.int32, device=dev)
+    slot_of = torch.tensor(list(range(n)) if decode else [0] * n, dtype=torch.int32, device=dev)
+    up = lambda a: torch.from_numpy(np.ascontiguousarray(a)).to(dev)
+    pairs = n * (context + 1) if decode else n * (n + 1) // 2
+    kp = (torch.randn(count * ppr, Ga, pt, hd, device=dev) * 0.5).bfloat16()
+    vp = (torch.randn(count * ppr, Ga, pt, hd, device=dev) * 0.5).bfloat16()
+    q = (torch.randn(n, Ha * hd, device=dev) * 0.5).bfloat16()
+    att = torch.empty(n, Ha * hd, dtype=bf, device=dev)
+    gate = torch.randn(n, Ha * hd, device=dev)
+    fixed = attention_fast.decode_splits(n, Ga, sm) if decode else 0
+    rws = 64 if decode else 256 if attention_fast.tc2_prefill_supported(hd, Ha // Ga, pt) else 128
+    plan = attention_fast.build_plan(slots, q_starts, q_lens, starts, n, 0, Ha, Ga, sm, up, fixed_splits=fixed,
+                                     max_context=context + 64 if decode else 0, prefill_rows=rws)
+    keys = (n * (context + 1) if decode else n) * Ga * hd * 4
+    dist = distance_table(torch.randn(32, Ha, device=dev), 1024)
+    dist2 = dist * math.log2(math.e)
+    us = _time_kernel(lambda: ops.paged_attention(q, kp, vp, table, positions, slot_of, att, Ha, Ga, hd, pt, 0, hd ** -0.5, plan=plan, gate=gate,
+                                                  dist=dist, dist_log2=dist2))
+    note("attention with distance bias and output gate", us, keys + n * Ha * hd * (4 + 4 + 4), 4.0 * pairs * Ha * hd, tc,
+         like="attention with soft cap and output gate (Mifolorn)")
+    us = _time_kernel(lambda: ops.paged_attention(q, kp, vp, table, positions, slot_of, att, Ha, Ga, hd, pt, 0, hd ** -0.5, plan=plan, gate=gate,
+                                                  softcap=50.0))
+    note("attention with soft cap and output gate (Mifolorn)", us, keys + n * Ha * hd * (4 + 4 + 4), 4.0 * pairs * Ha * hd, tc)
+    us = _time_kernel(lambda: ops.paged_attention(q, kp, vp, table, positions, slot_of, att, Ha, Ga, hd, pt, 0, hd ** -0.5, plan=plan, gate=gate))
+    note("attention with output gate alone", us, keys + n * Ha * hd * (4 + 4 + 4), 4.0 * pairs * Ha * hd, tc)
+    qkv = torch.randn(n, (Ha + 2 * Ga) * hd, device=dev)
+    bias = torch.zeros((Ha + 2 * Ga) * hd, device=dev)
+    qw, kw = torch.ones(Ha * hd, device=dev), torch.ones(Ga * hd, device=dev)
+    us = _time_kernel(lambda: ops.qk_row_norm_kv_write(qkv, q, qw, kw, Ha * hd, Ga * hd, 1e-6, positions, slot_of, table, kp, vp, Ha, Ga, hd, pt,
+                                                       bias=bias, q_factor=(0.3, 1024)))
+    note("qk_row_norm_kv_write (biases, query factor)", us, n * (Ha + 2 * Ga) * hd * 6, 0, 0,
+         like="qk_norm_rope_kv_write (Mifolorn: biases, half-rotated heads)")
+    cos, sin, qn = torch.ones(per + 1, 32, device=dev), torch.zeros(per + 1, 32, device=dev), torch.ones(hd, device=dev)
+    us = _time_kernel(lambda: ops.qk_norm_rope_kv_write(qkv, q, qn, qn, 1e-5, cos, sin, 64, positions, slot_of, table, kp, vp, Ha, Ga, hd, pt,
+                                                        bias=bias))
+    note("qk_norm_rope_kv_write (Mifolorn: biases, half-rotated heads)", us, n * (Ha + 2 * Ga) * hd * 6, 0, 0)
+
+    # ---- row-wise: the pair's normed sum with the next layer norm, layer norm, soft cap; the router
+    x, y, res = (torch.randn(n, width, device=dev) for _ in range(3))
+    xb = torch.empty(n, width, dtype=bf, device=dev)
+    w1, b1 = torch.ones(width, device=dev), torch.zeros(width, device=dev)
+    us = _time_kernel(lambda: ops.pair_norm_add(x, w1, 1e-6, 0.5, y, w1, 1e-6, 0.5, res, a_bias=b1, next_norm=(w1, b1, 1e-6), next_out=xb))
+    note("pair_norm_add (both results, bias, next layer norm)", us, n * width * (16 + 2), 0, 0, like="rms_norm_add")
+    us = _time_kernel(lambda: ops.rms_norm_add(x, w1, 1e-6, res))
+    note("rms_norm_add", us, n * width * 12, 0, 0)
+    us = _time_kernel(lambda: ops.layer_norm(x, w1, b1, 1e-6, xb))
+    note("layer_norm", us, n * width * 6, 0, 0, like="rms_norm")
+    us = _time_kernel(lambda: ops.rms_norm(x, w1, 1e-6, xb))
+    note("rms_norm", us, n * width * 6, 0, 0)
+    wanted = n if decode else 1
+    lgt = torch.randn(wanted, 32000, device=dev)
+    us = _time_kernel(lambda: ops.soft_cap(lgt, 30.0))
+    note("soft_cap of the logits", us, wanted * 32000 * 8, 0, 0, like="swiglu (as many numbers)")
+    gu = torch.randn(wanted, 32000, device=dev)
+    so = torch.empty(wanted, 16000, device=dev)
+    us = _time_kernel(lambda: ops.swiglu(gu, so))
+    note("swiglu (as many numbers)", us, wanted * 32000 * 4 + wanted * 16000 * 4, 0, 0)
+    E, top = 8, 2
+    wr, br, corr = torch.randn(E, width, device=dev) * 0.05, torch.randn(E, device=dev), torch.randn(E, device=dev) * 0.02
+    ids, wts = torch.empty(n, top, dtype=torch.int32, device=dev), torch.empty(n, top, device=dev)
+    us = _time_kernel(lambda: ops.route_topk(xb, wr, ids, wts, bias=br))
+    note("route_topk (softmax over the chosen, bias)", us, n * width * 2 + E * width * 4, 2.0 * n * E * width, fp32,
+         like="route_topk (Zazulix: sigmoid scores, groups)")
+    us = _time_kernel(lambda: ops.route_topk(xb, wr, ids, wts, "sigmoid", corr, 2, 1, 1.0, 1e-20))
+    note("route_topk (Zazulix: sigmoid scores, groups)", us, n * width * 2 + E * width * 4, 2.0 * n * E * width, fp32)
+    return out
+
+
 # design -> (its shape, the closest other design and its shape by width and layer runs)
 BESIDE = {"mifolorn": ("kedanex", lambda width, runs: kedanex_shape(width, runs // 4)),
           "zazulix": ("kedanex", lambda width, runs: kedanex_shape(width, runs // 4)),
-          "gezavik": ("zazulix", lambda width, runs: zazulix_shape(width, runs // 4))}
-SHAPES = {"kedanex": kedanex_shape, "padodra": padodra_shape, "mifolorn": mifolorn_shape, "zazulix": zazulix_shape, "gezavik": gezavik_shape}
+          "gezavik": ("zazulix", lambda width, runs: zazulix_shape(width, runs // 4)),
+          "nebanex": ("mifolorn", lambda width, runs: mifolorn_shape(width, runs // 4))}
+SHAPES = {"kedanex": kedanex_shape, "padodra": padodra_shape, "mifolorn": mifolorn_shape, "zazulix": zazulix_shape, "gezavik": gezavik_shape,
+          "nebanex": nebanex_shape}
 
 
 def run(design: str, args, peaks: dict) -> dict:
@@ -1000,6 +1154,9 @@ def run(design: str, args, peaks: dict) -> dict:
         elif design == "gezavik":
             entry["kernels_prefill_2048_rows"] = gezavik_kernel_points(width, 2048, False, peaks)
             entry["kernels_decode_64_rows"] = gezavik_kernel_points(width, 64, True, peaks)
+        elif design == "nebanex":
+            entry["kernels_prefill_2048_rows"] = nebanex_kernel_points(width, 2048, False, peaks)
+            entry["kernels_decode_64_rows"] = nebanex_kernel_points(width, 64, True, peaks)
         elif design == "kedanex":
             entry["kernels_prefill_2048_rows"] = kernel_points(width, 2048, peaks)
             entry["kernels_decode_64_rows"] = {k: v for k, v in kernel_points(width, 64, peaks).items() if "request" not in k or "decode" in k}
