@@ -47,6 +47,7 @@ LIBRARIES: Dict[str, str] = {
     "short_conv": "short_conv.cu",     # the causal convolution over a request's last rows that some mixers put behind their projections
     "state_space": "state_space.cu",   # the state-space recurrence (Mamba-2) and the gated norm behind it
     "gated_linear": "gated_linear.cu", # linear attention with a decay per key channel
+    "gated_linear_chunks": "gated_linear_chunks.cu",   # the same for prompt portions, chunks of tokens on the tensor cores
     "norms": "norms.cu",               # layer norm; two mixers' results normed onto the residual stream
     "routed": "routed.cu",             # a feed-forward of experts: route, sort, grouped products, combine
     "runtime": "runtime.cpp",          # host only: the cache's books (no GPU code, no CUDA headers)

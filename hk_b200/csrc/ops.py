@@ -987,11 +987,23 @@ def gla_decay(hid, w2, bias, tau: float, out) -> None:
                             ctypes.c_float(tau), _stream()), "gla_decay")
 
 
-def gla_scan(q, k, v, la, segments, state, out, n_heads: int, key_dim: int, value_dim: int, q_scale: float) -> None:
+GLA_CHUNK = 64      # tokens of a chunk of `gla_scan`'s chunked form
+
+
+def gla_chunks_take(key_dim: int, value_dim: int) -> bool:
+    """Whether the chunked form of `gla_scan` takes a mixer of these sizes."""
+    return key_dim % 8 == 0 and key_dim <= 128 and value_dim % 8 == 0
+
+
+def gla_scan(q, k, v, la, segments, state, out, n_heads: int, key_dim: int, value_dim: int, q_scale: float, chunks=None,
+             requests=None) -> None:
     """Linear attention with a decay per key channel over the rows of every segment, per head, S = state[slot, head] float32
     (stored [dv, dk]):
         S <- diag(2^la) S + k v^T;  out = S^T (q_scale q)
-    q, k [n, H*dk] and v [n, H*dv]: float32 column slices of ONE matrix; la float32 [n, H*dk]; out float32 [n, H*dv]."""
+    q, k [n, H*dk] and v [n, H*dv]: float32 column slices of ONE matrix; la float32 [n, H*dk]; out float32 [n, H*dv].
+    `chunks` int32 [n_chunks, 2] = (first row, rows) and `requests` int32 [n_requests, 3] = (slot, first chunk, chunks): further
+    requests that are walked in chunks of up to GLA_CHUNK tokens as matrix products on the tensor cores (sizes that
+    `gla_chunks_take`, 16-byte aligned slices); a request's chunks stand side by side, full ones first."""
     H, dk, dv = n_heads, key_dim, value_dim
     ld = _cols(q, "q", H * dk)
     if _cols(k, "k", H * dk) != ld or _cols(v, "v", H * dv) != ld:
@@ -1003,6 +1015,20 @@ def gla_scan(q, k, v, la, segments, state, out, n_heads: int, key_dim: int, valu
     n = q.shape[0]
     if tuple(state.shape[1:]) != (H, dv, dk) or tuple(out.shape) != (n, H * dv) or tuple(la.shape) != (n, H * dk) or segments.shape[1] != 3:
         raise KernelError("gla_scan: shapes do not fit")
+    if chunks is not None and chunks.shape[0]:
+        _need(chunks, "chunks", torch.int32, 2)
+        _need(requests, "requests", torch.int32, 2)
+        if chunks.shape[1] != 2 or requests.shape[1] != 3:
+            raise KernelError("gla_scan: chunks must be [n, 2] and requests [n, 3]")
+        nc = int(chunks.shape[0])
+        u = torch.empty(nc * H * dv * dk, dtype=torch.float32, device=out.device)
+        decay = torch.empty(nc * H * dk, dtype=torch.float32, device=out.device)
+        lib = build.load("gated_linear_chunks")
+        _check(lib.hk_gla_chunks(_ptr(q), _ptr(k), _ptr(v), ctypes.c_longlong(ld), _ptr(la), _ptr(chunks), nc, _ptr(requests),
+                                 int(requests.shape[0]), _ptr(u), _ptr(decay), _ptr(state), _ptr(out), H, dk, dv, ctypes.c_float(q_scale),
+                                 _stream()), "gla_scan (chunks)", launches=3)
+    if not segments.shape[0]:
+        return
     lib = build.load("gated_linear")
     _check(lib.hk_gla_walk(_ptr(q), _ptr(k), _ptr(v), ctypes.c_longlong(ld), _ptr(la), _ptr(segments), int(segments.shape[0]),
                            _ptr(state), _ptr(out), H, dk, dv, ctypes.c_float(q_scale), 1 if segments.shape[0] == n else 0, _stream()),

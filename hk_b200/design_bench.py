@@ -1016,11 +1016,33 @@ def nebanex_kernel_points(width: int, n: int, decode: bool, peaks: dict) -> dict
     ab = torch.full((K,), 2.0, device=dev)
     la = torch.empty(n, K, device=dev)
     us = _time_kernel(lambda: ops.gla_decay(proj[:, 2 * K + 2 * V:], w2, ab, 16.0, la))
-    note("gla_decay (low-rank logits to log decays)", us, n * (R + K) * 4 + K * (R + 1) * 4, 2.0 * n * K * R, fp32, like="rms_norm")
+    note("gla_decay (low-rank logits to log decays)", us, n * (R + K) * 4 + K * (R + 1) * 4, 2.0 * n * K * R, fp32,
+         like="tanh and second product of a low-rank decay (Kedanex)")
+    hid = torch.empty(n, R, dtype=bf, device=dev)
+    w2b = w2.bfloat16()
+
+    def low_rank():
+        ops.tanh_cols(proj[:, 2 * K + 2 * V:], hid)
+        ops.gemm(hid, w2b, la)
+
+    us = _time_kernel(low_rank)
+    note("tanh and second product of a low-rank decay (Kedanex)", us, n * (R + K) * 4 + K * R * 2, 2.0 * n * K * R, fp32)
+    us = _time_kernel(lambda: ops.gla_decay(proj[:, 2 * K + 2 * V:], w2, ab, 16.0, la))      # the values the scan reads
     state = torch.zeros(count, H, dv, dk, device=dev)
     o = torch.empty(n, V, device=dev)
-    us = _time_kernel(lambda: ops.gla_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], la, sg, state, o, H, dk, dv, dk ** -0.5))
-    note("gla_scan", us, 4 * (n * (3 * K + 2 * V) + 2 * count * H * dk * dv), 5.0 * n * H * dk * dv, fp32, like="gated_delta_scan (Mifolorn)")
+    walk = lambda: ops.gla_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], la, sg, state, o, H, dk, dv, dk ** -0.5)
+    moved = 4 * (n * (3 * K + 2 * V) + 2 * count * H * dk * dv)
+    if decode:
+        us = _time_kernel(walk)
+        note("gla_scan", us, moved, 5.0 * n * H * dk * dv, fp32, like="gated_delta_scan (Mifolorn)")
+    else:       # a prompt's chunks run on the tensor cores, where the bytes are the floor
+        chunks = torch.tensor([[t, min(ops.GLA_CHUNK, n - t)] for t in range(0, n, ops.GLA_CHUNK)], dtype=torch.int32, device=dev)
+        reqs = torch.tensor([[0, 0, chunks.shape[0]]], dtype=torch.int32, device=dev)
+        us = _time_kernel(lambda: ops.gla_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], la, sg[:0], state, o, H, dk, dv,
+                                               dk ** -0.5, chunks, reqs))
+        note("gla_scan", us, moved, 5.0 * n * H * dk * dv, tc, like="gated_delta_scan (Mifolorn)")
+        us = _time_kernel(walk)
+        note("gla_scan, token by token", us, moved, 5.0 * n * H * dk * dv, fp32, like="gated_delta_scan (Mifolorn)")
     Hd, Gd = width // 64, width // 128
     Kd, Vd = Gd * 64, Hd * 64
     act = torch.randn(n, 2 * Kd + Vd, device=dev) * 0.5

@@ -66,10 +66,10 @@ class ParallelMixer(Part):
     def bind(self, tensors, precision) -> None:
         super().bind(tensors, precision)
         if self._stacked:           # the sides' own copies become views of the one matrix
-            n_left = int(self.left.in_weight.shape[0])
-            n_right = int(self.right.in_weight.shape[0])
-            self.w_in = stacked_rows([self.left.in_weight, self.right.in_weight], multiple=8)
-            self.left.in_weight, self.right.in_weight = self.w_in[:n_left], self.w_in[n_left:n_left + n_right]
+            n_left, n_right = int(self.left.in_weight.shape[0]), int(self.right.in_weight.shape[0])
+            self.w_in = stacked_rows([stacked_rows([self.left.in_weight], multiple=8), self.right.in_weight], multiple=8)
+            at = -(-n_left // 8) * 8            # both sides' columns start aligned for wide loads
+            self.left.in_weight, self.right.in_weight = self.w_in[:n_left], self.w_in[at:at + n_right]
 
     def takes_next_norm(self, norm) -> bool:
         """Whether `forward` can write the layer norm of the new residual stream as well (`next_norm`, `next_out`)."""
@@ -85,8 +85,9 @@ class ParallelMixer(Part):
         if self._stacked:
             proj = torch.empty((xb.shape[0], self.w_in.shape[0]), dtype=torch.float32, device=xb.device)
             ops.gemm(xb, self.w_in, proj)
-            n_left = self.left.in_weight.shape[0]
-            left_more["proj"], right_more["proj"] = proj[:, :n_left], proj[:, n_left:]
+            n_left, n_right = self.left.in_weight.shape[0], self.right.in_weight.shape[0]
+            at = -(-n_left // 8) * 8
+            left_more["proj"], right_more["proj"] = proj[:, :n_left], proj[:, at:at + n_right]
         if self._carried:
             self.left.forward(xb, residual, ctx, left_cache, write_cache, accumulate=accumulate, **left_more)
             self.right.forward(xb, residual, ctx, right_cache, write_cache, accumulate=True, **right_more)

@@ -443,8 +443,12 @@ class StateSpace(_SegmentScan):
 
 
 class GatedLinearAttention(_SegmentScan):
-    kernel_libraries = ("gated_linear", "recurrent")
+    """When serving in bfloat16, a request that brings `CHUNKS_FROM` tokens or more to a step is walked in chunks of tokens on
+    the tensor cores (`ops.gla_scan`), the others token by token; the lists of requests and chunks are this part's host-built
+    tables."""
     takes_projection = True     # `forward` can be handed the product with `in_weight` (`proj`)
+    CHUNKS_FROM = 64
+    SPLIT_KEY = ("gated_linear_segments",)
 
     def __init__(self, hidden: int, n_heads: int, key_dim: int, value_dim: int, tau: float, prefix: str, norm_eps: float,
                  decay_rank: Optional[int] = None, q_scale: Optional[float] = None, names: Optional[Dict[str, str]] = None):
@@ -458,6 +462,28 @@ class GatedLinearAttention(_SegmentScan):
         self.names.update(names or {})
         self.in_weight = self.w_o = self.w_a2 = self.a_bias = self.norm_weight = None
         self.rank = 0
+        self._chunks = False            # set at bind: the chunked walk takes this mixer's sizes
+
+    def kernel_libraries(self, bfloat16: bool):
+        chunked = bfloat16 and ops.gla_chunks_take(self.dk, self.dv)
+        return ("gated_linear", "recurrent") + (("gated_linear_chunks",) if chunked else ())
+
+    def step_tables_key(self):
+        return self.SPLIT_KEY if self._chunks else SEGMENTS_KEY
+
+    def step_tables(self, ctx):
+        tables = segment_tables(ctx)
+        if not self._chunks:
+            return tables
+        seg = tables.arrays["segments"]
+        long = seg[:, 2] >= self.CHUNKS_FROM
+        chunks, requests = [], []
+        for slot, row, count in seg[long].tolist():
+            first = len(chunks)
+            chunks += [(row + t, min(ops.GLA_CHUNK, count - t)) for t in range(0, count, ops.GLA_CHUNK)]
+            requests.append((slot, first, len(chunks) - first))
+        return StepTables({"short": seg[~long], "chunks": np.asarray(chunks, dtype=np.int32).reshape(-1, 2),
+                           "requests": np.asarray(requests, dtype=np.int32).reshape(-1, 3)})
 
     def own_param_specs(self) -> Dict[str, ParamSpec]:
         p, nm, d = self.prefix, self.names, self.hidden
@@ -476,12 +502,13 @@ class GatedLinearAttention(_SegmentScan):
     def own_bind(self, tensors, precision: Precision) -> None:
         p, nm = self.prefix, self.names
         # one product gives q, k, v, the output gate's logits and the hidden layer of the decay's low-rank projection
-        self.in_weight = stacked_rows([tensors[p + nm[c]] for c in ("q", "k", "v", "g", "a1")])
+        self.in_weight = stacked_rows([tensors[p + nm[c]] for c in ("q", "k", "v", "g", "a1")], multiple=8)
         self.rank = int(tensors[p + nm["a1"]].shape[0])
         self.w_a2, self.a_bias = tensors[p + nm["a2"]], tensors[p + nm["a_bias"]]
         if int(self.w_a2.shape[1]) != self.rank:
             raise ValueError(f"'{p + nm['a2']}' takes {int(self.w_a2.shape[1])} inputs, '{p + nm['a1']}' gives {self.rank}")
         self.w_o, self.norm_weight = tensors[p + nm["o"]], tensors[p + nm["norm"]]
+        self._chunks = precision.compute == torch.bfloat16 and ops.gla_chunks_take(self.dk, self.dv)
 
     def forward(self, xb: torch.Tensor, residual: torch.Tensor, ctx, cache, write_cache: bool = True,
                 accumulate: bool = True, proj=None) -> None:
@@ -495,8 +522,9 @@ class GatedLinearAttention(_SegmentScan):
         la = torch.empty((n, K), dtype=torch.float32, device=dev)
         ops.gla_decay(proj[:, a0:a0 + self.rank], self.w_a2, self.a_bias, self.tau, la)
         o = torch.empty((n, V), dtype=torch.float32, device=dev)
-        ops.gla_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], la, self._segments(ctx), cache.state, o, H, self.dk,
-                     self.dv, self.q_scale)
+        arrays = ctx.tables[self.step_tables_key()][0]
+        ops.gla_scan(proj[:, :K], proj[:, K:2 * K], proj[:, 2 * K:2 * K + V], la, arrays["short" if self._chunks else "segments"],
+                     cache.state, o, H, self.dk, self.dv, self.q_scale, arrays.get("chunks"), arrays.get("requests"))
         og = torch.empty((n, V), dtype=xb.dtype, device=dev)
         ops.head_out_gate(o, proj[:, 2 * K + V:a0], self.norm_weight, self.norm_eps, og, H, self.dv, act="silu")
         ops.gemm(og, self.w_o, residual, accumulate=accumulate)

@@ -144,6 +144,8 @@ LINEAR = [
     (24, 1, 21, 34, 1.0, 1),         # tau of 1: decays that forget at once
     (24, 2, 200, 6, 2.0, 9),         # keys that end inside a lane's share, above 128
     (24, 1, 264, 3, 3.0, 2),
+    (32, 2, 24, 136, 2.0, 3),        # more value columns than a block of the chunked walk; keys that end inside a tile
+    (40, 1, 96, 64, 6.0, 4),
 ]
 
 
@@ -173,6 +175,25 @@ def test_gated_linear_long_portions_beside_single_tokens(dtype, dk, dv, tau):
         got = hs.run(steps)
         for r in lengths:
             close(got[r], want[r], dtype, r)
+
+
+@pytest.mark.parametrize("dk,dv", [(64, 128), (32, 48), (128, 16)])
+def test_gated_linear_chunks_of_several_long_requests(dk, dv):
+    """Portions of many chunks (more than the carry asks for at once) of three requests in one batch, beside a short one, against
+    the walk token by token of the same part."""
+    part, prec, w, m = gated_linear(40, 2, dk, dv, 8.0, 6, torch.bfloat16)
+    lengths = {"a": 1290, "b": 640, "c": 700}
+    x = {r: torch.randn(n, 40, device="cuda").to(torch.bfloat16) for r, n in lengths.items()}
+    hs = Harness(part, prec, torch.bfloat16, x)
+    steps = [[("a", 1088), ("b", 3), ("c", 65)], [("c", 571), ("a", 1), ("b", 637)], [("a", 201), ("c", 64)]]
+    assert part._chunks
+    got = hs.run(steps)
+    part._chunks = False
+    want = hs.run(steps)
+    for r in lengths:
+        close(got[r], want[r], torch.bfloat16, r)
+    plain = P.gated_linear(x["b"].double().cpu().numpy(), w, "m.", m, 1e-5)
+    close(got["b"], plain, torch.bfloat16, "plain")
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
@@ -229,10 +250,8 @@ def test_pair_of_mixers_with_normed_results(dtype, d):
     for part in (left_out, right_out, norm):
         w.update(bind_random(part, dtype, seed=3, std=0.3)[1])
     pair = ParallelMixer(left, right, 0.5, 0.25, left_out, right_out)
-    n_left = left.in_weight.shape[0]
-    from hk_b200.parts.base import stacked_rows
-    pair.w_in = stacked_rows([left.in_weight, right.in_weight], multiple=8)
-    left.in_weight, right.in_weight = pair.w_in[:n_left], pair.w_in[n_left:n_left + right.in_weight.shape[0]]
+    left.bind = right.bind = left_out.bind = right_out.bind = lambda tensors, precision: None      # bound above, and changed since
+    pair.bind({}, prec)
 
     def plain(x):
         a = P.rms(P.attention(x, w, "m.left.", ml, 1e-5), 1e-5) * w["m.left.out"]
