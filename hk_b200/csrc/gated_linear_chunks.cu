@@ -123,29 +123,41 @@ gla_states_kernel(const float* __restrict__ k, const float* __restrict__ v, long
   const int col0 = blockIdx.y * DVB, ncols = min(DVB, dv - col0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int e = tid; e < CQ * (NT / 4); e += NTH) {
-    const int t = e / (NT / 4), i = (e % (NT / 4)) * 4;
-    *reinterpret_cast<float4*>(b + t * K::LB + i) =
-        t < ch.count && i < dk ? *reinterpret_cast<const float4*>(la + ((size_t)(ch.row0 + t) * H + h) * dk + i) : zero;
+  // everything is asked for at once; the keys wait in registers for the cumulative decays
+  constexpr int NK = CQ * (NT / 4) / NTH, NV = CQ * (DVB / 4) / NTH;
+  float4 kr[NK], lr[NK], vr[NV];
+#pragma unroll
+  for (int j = 0; j < NK; ++j) {
+    const int e = tid + j * NTH, t = e / (NT / 4), i = (e % (NT / 4)) * 4;
+    const bool in = t < ch.count && i < dk;
+    lr[j] = in ? *reinterpret_cast<const float4*>(la + ((size_t)(ch.row0 + t) * H + h) * dk + i) : zero;
+    kr[j] = in ? *reinterpret_cast<const float4*>(k + (size_t)(ch.row0 + t) * ld + (size_t)h * dk + i) : zero;
   }
-  for (int e = tid; e < CQ * (DVB / 4); e += NTH) {
-    const int t = e / (DVB / 4), d = (e % (DVB / 4)) * 4;
-    const float4 x = t < ch.count && d < ncols ? *reinterpret_cast<const float4*>(v + (size_t)(ch.row0 + t) * ld + (size_t)h * dv + col0 + d) : zero;
-    *reinterpret_cast<uint2*>(vs + t * K::LV + d) = make_uint2(pack(x.x, x.y), pack(x.z, x.w));
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int e = tid + j * NTH, t = e / (DVB / 4), d = (e % (DVB / 4)) * 4;
+    vr[j] = t < ch.count && d < ncols ? *reinterpret_cast<const float4*>(v + (size_t)(ch.row0 + t) * ld + (size_t)h * dv + col0 + d) : zero;
+  }
+#pragma unroll
+  for (int j = 0; j < NK; ++j) {
+    const int e = tid + j * NTH;
+    *reinterpret_cast<float4*>(b + (e / (NT / 4)) * K::LB + (e % (NT / 4)) * 4) = lr[j];
+  }
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int e = tid + j * NTH;
+    *reinterpret_cast<uint2*>(vs + (e / (DVB / 4)) * K::LV + (e % (DVB / 4)) * 4) = make_uint2(pack(vr[j].x, vr[j].y), pack(vr[j].z, vr[j].w));
   }
   __syncthreads();
   cumulate<NT, K::LB>(b, tot);
   const float* last = b + (CQ - 1) * K::LB;
   if (blockIdx.y == 0)
     for (int i = tid; i < dk; i += NTH) decay[((size_t)c * H + h) * dk + i] = exp2_f(last[i]);
-  for (int e = tid; e < CQ * (NT / 4); e += NTH) {
-    const int t = e / (NT / 4), i = (e % (NT / 4)) * 4;
-    float4 x = zero;
-    if (t < ch.count && i < dk) {
-      x = *reinterpret_cast<const float4*>(k + (size_t)(ch.row0 + t) * ld + (size_t)h * dk + i);
-      const float4 z = *reinterpret_cast<const float4*>(last + i), y = *reinterpret_cast<const float4*>(b + t * K::LB + i);
-      x = make_float4(x.x * exp2_f(z.x - y.x), x.y * exp2_f(z.y - y.y), x.z * exp2_f(z.z - y.z), x.w * exp2_f(z.w - y.w));
-    }
+#pragma unroll
+  for (int j = 0; j < NK; ++j) {
+    const int e = tid + j * NTH, t = e / (NT / 4), i = (e % (NT / 4)) * 4;
+    const float4 x0 = kr[j], z = *reinterpret_cast<const float4*>(last + i), y = *reinterpret_cast<const float4*>(b + t * K::LB + i);
+    const float4 x = make_float4(x0.x * exp2_f(z.x - y.x), x0.y * exp2_f(z.y - y.y), x0.z * exp2_f(z.z - y.z), x0.w * exp2_f(z.w - y.w));
     uint32_t lo[3], hi[3];
     split3(x.x, x.y, lo);
     split3(x.z, x.w, hi);
@@ -278,6 +290,7 @@ gla_out_kernel(const float* __restrict__ q, const float* __restrict__ k, const f
       }
   }
 
+#pragma unroll 4
   for (int e = tid; e < CQ * C4; e += NTH) {
     const int t = e / C4, i = (e % C4) * 4;
     const bool in = t < ch.count && i < dk;

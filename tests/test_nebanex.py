@@ -131,13 +131,13 @@ def test_gated_linear_tables_part_long_requests_from_short_ones():
 
     from hk_b200.parts import GatedLinearAttention
     part = GatedLinearAttention(16, 2, 8, 8, 2.0, "m.", 1e-5)
-    ctx = SimpleNamespace(slots=[4, 1, 0, 2], q_starts=[0, 63, 127, 128], q_lens=[63, 64, 1, 150])
-    np.testing.assert_array_equal(part.step_tables(ctx).arrays["segments"], [[4, 0, 63], [1, 63, 64], [0, 127, 1], [2, 128, 150]])
+    ctx = SimpleNamespace(slots=[4, 1, 0, 2], q_starts=[0, 127, 255, 256], q_lens=[127, 128, 1, 150])
+    np.testing.assert_array_equal(part.step_tables(ctx).arrays["segments"], [[4, 0, 127], [1, 127, 128], [0, 255, 1], [2, 256, 150]])
     part._chunks = True
     arrays = part.step_tables(ctx).arrays
-    np.testing.assert_array_equal(arrays["short"], [[4, 0, 63], [0, 127, 1]])
-    np.testing.assert_array_equal(arrays["chunks"], [[63, 64], [128, 64], [192, 64], [256, 22]])
-    np.testing.assert_array_equal(arrays["requests"], [[1, 0, 1], [2, 1, 3]])
+    np.testing.assert_array_equal(arrays["short"], [[4, 0, 127], [0, 255, 1]])
+    np.testing.assert_array_equal(arrays["chunks"], [[127, 64], [191, 64], [256, 64], [320, 64], [384, 22]])
+    np.testing.assert_array_equal(arrays["requests"], [[1, 0, 2], [2, 2, 3]])
     ctx = SimpleNamespace(slots=[3], q_starts=[0], q_lens=[1])
     arrays = part.step_tables(ctx).arrays
     assert arrays["chunks"].shape == (0, 2) and arrays["requests"].shape == (0, 3) and arrays["short"].shape == (1, 3)

@@ -171,8 +171,9 @@ def test_gated_linear_long_portions_beside_single_tokens(dtype, dk, dv, tau):
     hs = Harness(part, prec, dtype, x)
     steps = [[("a", 31), ("b", 1)], [("b", 32), ("a", 1), ("c", 2)], [("a", 64), ("c", 1), ("b", 2)], [("b", 65), ("a", 63)],
              [("a", 66), ("b", 33), ("c", 35)], [("a", 2), ("b", 1), ("c", 2)], [("a", 33)], [("b", 16)]]
-    for _ in range(2):
-        got = hs.run(steps)
+    long = [[("a", 129), ("c", 1)], [("b", 150), ("a", 131), ("c", 39)]]
+    for st in (steps, long, steps):
+        got = hs.run(st)
         for r in lengths:
             close(got[r], want[r], dtype, r)
 
