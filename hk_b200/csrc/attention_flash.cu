@@ -589,7 +589,8 @@ __device__ __forceinline__ void tma_load_3d(void* dst, const CUtensorMap* map, u
       ::"r"(smem_u32(dst)), "l"(map), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2) : "memory");
 }
 
-template <int HD>
+// DIST: with a bias by distance (an instance of its own, so that the steps of a model without one issues nothing for it)
+template <int HD, bool DIST>
 __global__ void __launch_bounds__((TW + 1) * 32, 2)
 attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                             const bf16* __restrict__ q, const int* __restrict__ block_table, int table_stride,
@@ -683,7 +684,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
       lo[i] = window > 0 ? max(0, pos[i] - window + 1) : 0;
     if (so.chunk > 0) lo[i] = max(lo[i], (pos[i] / so.chunk) * so.chunk);
       qp[i] = q + ((size_t)(it.q_row0 + tq) * H + g * group + row[i] % group) * HD;
-      drow[i] = so.dist ? so.dist + (size_t)(g * group + row[i] % group) * so.dist_n : nullptr;
+      drow[i] = DIST ? so.dist + (size_t)(g * group + row[i] % group) * so.dist_n : nullptr;
     }
     uint32_t qf[KSTEPS][4];
 #pragma unroll
@@ -735,7 +736,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
           const int i = e >> 1;
           const int j = t * TT + warp * 16 + nn * 8 + 2 * qt + (e & 1);
           const bool ok = valid[i] && j >= lo[i] && j <= pos[i] && j >= it.kv_lo && j < it.kv_hi;
-          s[nn][e] = ok ? scaled_score(s[nn][e], scale_log2, so) + (so.dist ? distance_bias(drow[i], pos[i] - j, so) : 0.f) : -CUDART_INF_F;
+          s[nn][e] = ok ? scaled_score(s[nn][e], scale_log2, so) + (DIST ? distance_bias(drow[i], pos[i] - j, so) : 0.f) : -CUDART_INF_F;
           mt[i] = fmaxf(mt[i], s[nn][e]);
         }
       float corr[2], msafe[2];
@@ -1021,16 +1022,16 @@ bool make_page_map(CUtensorMap* map, const void* ptr, unsigned long long rows, i
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int HD>
+template <int HD, bool DIST>
 int launch_decode_tma(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, const int* bt, int stride, const void* items,
                       int n_items, void* out, float* part_o, float* part_ml, int H, int G, int pt, int box_rows, int window,
                       float scale_log2, ScoreOpts so, int pages_cap, int* status, cudaStream_t s) {
   const size_t smem = 1024 + (size_t)2 * TS * TT * HD * 2 + 2 * TS * sizeof(uint64_t) + 8 + (size_t)pages_cap * sizeof(int);
   if (smem > 110 * 1024) return HK_ERR_UNSUPPORTED;
   static HkSmemCache allowed = {};
-  if (int e = hk_allow_smem(attention_decode_tma_kernel<HD>, smem, allowed)) return e;
+  if (int e = hk_allow_smem(attention_decode_tma_kernel<HD, DIST>, smem, allowed)) return e;
   dim3 grid((unsigned)n_items, (unsigned)G);
-  return hk_launch_pdl(attention_decode_tma_kernel<HD>, grid, dim3((TW + 1) * 32), smem, s, mk, mv, (const bf16*)q, bt, stride,
+  return hk_launch_pdl(attention_decode_tma_kernel<HD, DIST>, grid, dim3((TW + 1) * 32), smem, s, mk, mv, (const bf16*)q, bt, stride,
                        (const Item*)items, (bf16*)out, part_o, part_ml, H, G, pt, box_rows, window, scale_log2, so, pages_cap, status);
 }
 
@@ -1054,11 +1055,12 @@ HK_API int hk_attention_decode_tma(const void* q, const void* k_pages, const voi
   CUtensorMap mk, mv;
   if (!make_page_map(&mk, k_pages, rows, hd, box_rows) || !make_page_map(&mv, v_pages, rows, hd, box_rows)) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
-  if (hd == 64)
-    return launch_decode_tma<64>(mk, mv, q, block_table, table_stride, items, n_items, out, part_o, part_ml, H, G, page_tokens,
-                                 box_rows, window, scale_log2, so, pages_cap, status, s);
-  return launch_decode_tma<128>(mk, mv, q, block_table, table_stride, items, n_items, out, part_o, part_ml, H, G, page_tokens,
-                                box_rows, window, scale_log2, so, pages_cap, status, s);
+#define HK_TMA(D, WITH)                                                                                                      \
+  launch_decode_tma<D, WITH>(mk, mv, q, block_table, table_stride, items, n_items, out, part_o, part_ml, H, G, page_tokens, \
+                             box_rows, window, scale_log2, so, pages_cap, status, s)
+  if (hd == 64) return so.dist ? HK_TMA(64, true) : HK_TMA(64, false);
+  return so.dist ? HK_TMA(128, true) : HK_TMA(128, false);
+#undef HK_TMA
 }
 
 // ---- the entry point that allocates nothing (see attention_noalloc.h) -------------------------------------

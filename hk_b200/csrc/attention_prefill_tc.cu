@@ -232,7 +232,8 @@ struct Smem {
   int pages[1];        // [pages_cap], the tail of the dynamic allocation: page ids of the item's key range
 };
 
-template <int HD>
+// DIST: with a bias by distance (an instance of its own, so that the softmax of a model without one issues nothing for it)
+template <int HD, bool DIST>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                             const int* __restrict__ block_table, int table_stride, const Item* __restrict__ items,
@@ -431,8 +432,8 @@ attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__
     const float sl = so.cap_log2 > 0.f ? 1.0f : scale_log2;      // capped scores are in the exponent's domain already
     const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
     constexpr int HK = TK / 2, HO = HD / 2;          // keys and O columns per thread
-    const float* drow = so.dist ? so.dist + (size_t)(g * group + (valid ? r % group : 0)) * so.dist_n : nullptr;
-    const float far_bias = drow ? drow[so.dist_n - 1] : 0.f;
+    const float* drow = DIST && so.dist ? so.dist + (size_t)(g * group + (valid ? r % group : 0)) * so.dist_n : nullptr;
+    const float far_bias = DIST && drow ? drow[so.dist_n - 1] : 0.f;
     float m = -CUDART_INF_F, l = 0.f;
     bool ok = true;
     for (int t = t_begin; t < t_end; ++t) {
@@ -466,14 +467,14 @@ attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__
       // than the table reaches, their bias is one number and rides on the maximum and the exponent's constant; else every
       // score takes its own.
       float slt = sl, add = far_bias;
-      if (drow && pos - (j0 + HK - 1) < so.dist_n - 1) {
+      if (DIST && drow && pos - (j0 + HK - 1) < so.dist_n - 1) {
         add_distance_bias<HK>(su, drow, pos - j0, sl, so.dist_n);
         slt = 1.0f;
         add = 0.f;
       }
 #pragma unroll
       for (int i = 0; i < HK; ++i) mraw = fmaxf(mraw, __uint_as_float(su[i]));
-      mraw = fmaf(mraw, slt, add);
+      mraw = DIST ? fmaf(mraw, slt, add) : mraw * slt;
       sm.xmax[n & 1][half][r] = mraw;
       asm volatile("bar.sync %0, 64;" ::"r"(1 + quarter) : "memory");     // the two warps of this quarter
       mraw = fmaxf(mraw, sm.xmax[n & 1][half ^ 1][r]);
@@ -495,11 +496,12 @@ attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__
       const int need = any_move ? n - 1 : n - 2;     // the P V product that has to be complete by now
       if (need >= 0 && !__all_sync(0xffffffffu, mbar_wait(&sm.pv_done[need & 1], (uint32_t)((need >> 1) & 1), abort_flag))) { ok = false; break; }
       tc_fence_after();
+      const float shift = DIST ? add - msafe : -msafe;
       uint32_t pw[HK / 2];
 #pragma unroll
       for (int e = 0; e < HK / 2; ++e) {
-        const float p0 = ex2(fmaf(__uint_as_float(su[2 * e]), slt, add - msafe));
-        const float p1 = ex2(fmaf(__uint_as_float(su[2 * e + 1]), slt, add - msafe));
+        const float p0 = ex2(fmaf(__uint_as_float(su[2 * e]), slt, shift));
+        const float p1 = ex2(fmaf(__uint_as_float(su[2 * e + 1]), slt, shift));
         l += p0 + p1;
         __nv_bfloat162 pk = __floats2bfloat162_rn(p0, p1);
         pw[e] = *reinterpret_cast<uint32_t*>(&pk);
@@ -557,15 +559,15 @@ attention_prefill_tc_kernel(const bf16* __restrict__ q, const bf16* __restrict__
   }
 }
 
-template <int HD>
+template <int HD, bool DIST>
 int launch(const void* q, const void* kp, const void* vp, const int* bt, int stride, const void* items, int n_items, void* out,
            int H, int G, int pt, int window, float scale_log2, ScoreOpts so, int pages_cap, int* status, cudaStream_t s) {
   const size_t smem = sizeof(Smem<HD>) + 1024 + (size_t)pages_cap * sizeof(int);
   if (smem > 225 * 1024) return HK_ERR_UNSUPPORTED;
   static HkSmemCache allowed = {};
-  if (int e = hk_allow_smem(attention_prefill_tc_kernel<HD>, smem, allowed)) return e;
+  if (int e = hk_allow_smem(attention_prefill_tc_kernel<HD, DIST>, smem, allowed)) return e;
   dim3 grid((unsigned)n_items * (unsigned)G);
-  attention_prefill_tc_kernel<HD><<<grid, NUM_THREADS, smem, s>>>((const bf16*)q, (const bf16*)kp, (const bf16*)vp, bt, stride,
+  attention_prefill_tc_kernel<HD, DIST><<<grid, NUM_THREADS, smem, s>>>((const bf16*)q, (const bf16*)kp, (const bf16*)vp, bt, stride,
                                                                  (const Item*)items, (bf16*)out, H, G, pt, window, scale_log2,
                                                                  so, pages_cap, status);
   return hk_launch_status();
@@ -615,7 +617,8 @@ struct Smem2 {
   int pages[1];        // [pages_cap]
 };
 
-template <int HD>
+// DIST: with a bias by distance (an instance of its own, so that the softmax of a model without one issues nothing for it)
+template <int HD, bool DIST>
 __global__ void __launch_bounds__(NT2, 1)
 attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                              const bf16* __restrict__ q, const int* __restrict__ block_table, int table_stride,
@@ -791,8 +794,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
     cp_async_wait<0>();
     fence_async_proxy();
     mbar_arrive(&sm.q_full);
-    const float* drow = so.dist ? so.dist + (size_t)(g * group + (valid ? row % group : 0)) * so.dist_n : nullptr;
-    const float far_bias = drow ? drow[so.dist_n - 1] : 0.f;
+    const float* drow = DIST && so.dist ? so.dist + (size_t)(g * group + (valid ? row % group : 0)) * so.dist_n : nullptr;
+    const float far_bias = DIST && drow ? drow[so.dist_n - 1] : 0.f;
     float m = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
     bool ok = true;
     if (qt == 0 || two) {
@@ -829,7 +832,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
           }
           // keys further back than the table reaches share one bias, which rides on the exponent's constant
           float slt = sl, add = far_bias;
-          if (drow && pos - (j0 + 32 * c + 31) < so.dist_n - 1) {
+          if (DIST && drow && pos - (j0 + 32 * c + 31) < so.dist_n - 1) {
             add_distance_bias<32>(su, drow, pos - (j0 + 32 * c), sl, so.dist_n);
             slt = 1.0f;
             add = 0.f;
@@ -840,7 +843,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
 #pragma unroll
             for (int e = 0; e < 4; ++e) mx[e] = fmaxf(mx[e], fmaxf(__uint_as_float(su[i + 2 * e]), __uint_as_float(su[i + 2 * e + 1])));
           }
-          const float cm = fmaf(fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])), slt, add);
+          const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+          const float cm = DIST ? fmaf(top, slt, add) : top * slt;
           const bool move = cm > m + 8.0f;
           if (__any_sync(0xffffffffu, move)) {
             const float mn = move ? ceilf(cm) : m;
@@ -875,7 +879,8 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __
             }
             m = mn;
           }
-          const float shift = add - (m == -CUDART_INF_F ? 0.f : m);
+          const float msafe = m == -CUDART_INF_F ? 0.f : m;
+          const float shift = DIST ? add - msafe : -msafe;
           uint32_t pw[16];
 #pragma unroll
           for (int e = 0; e < 16; ++e) {
@@ -955,15 +960,15 @@ bool make_page_map(CUtensorMap* map, const void* ptr, unsigned long long rows, i
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int HD>
+template <int HD, bool DIST>
 int launch2(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, const int* bt, int stride, const void* items, int n_items,
             void* out, int H, int G, int pt, int window, float scale_log2, ScoreOpts so, int pages_cap, int* status, cudaStream_t s) {
   const size_t smem = sizeof(Smem2<HD>) + 1024 + (size_t)pages_cap * sizeof(int);
   if (smem > 225 * 1024) return HK_ERR_UNSUPPORTED;
   static HkSmemCache allowed = {};
-  if (int e = hk_allow_smem(attention_prefill_tc2_kernel<HD>, smem, allowed)) return e;
+  if (int e = hk_allow_smem(attention_prefill_tc2_kernel<HD, DIST>, smem, allowed)) return e;
   dim3 grid((unsigned)n_items * (unsigned)G);
-  return hk_launch(attention_prefill_tc2_kernel<HD>, grid, dim3(NT2), smem, s, mk, mv, (const bf16*)q, bt, stride, (const Item*)items,
+  return hk_launch(attention_prefill_tc2_kernel<HD, DIST>, grid, dim3(NT2), smem, s, mk, mv, (const bf16*)q, bt, stride, (const Item*)items,
                    (bf16*)out, H, G, pt, window, scale_log2, so, pages_cap, status);
 }
 
@@ -998,8 +1003,10 @@ HK_API int hk_attention_prefill_tc(const void* q, const void* k_pages, const voi
   if (G < 1 || H % G != 0 || (H / G) > ROWS || G > 65535 || page_tokens < 1 || !(scale_log2 > 0.f)) return HK_ERR_UNSUPPORTED;
   if ((((uintptr_t)q | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)out) & 15) != 0) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
-  if (hd == 128) return launch<128>(q, k_pages, v_pages, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
-  if (hd == 64) return launch<64>(q, k_pages, v_pages, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
+  if (hd == 128) return so.dist ? launch<128, true>(q, k_pages, v_pages, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s)
+                       : launch<128, false>(q, k_pages, v_pages, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
+  if (hd == 64) return so.dist ? launch<64, true>(q, k_pages, v_pages, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s)
+                       : launch<64, false>(q, k_pages, v_pages, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
   return HK_ERR_UNSUPPORTED;
 }
 
@@ -1024,7 +1031,9 @@ HK_API int hk_attention_prefill_tc2(const void* q, const void* k_pages, const vo
   CUtensorMap mk, mv;
   if (!make_page_map(&mk, k_pages, rows, hd, box_rows) || !make_page_map(&mv, v_pages, rows, hd, box_rows)) return HK_ERR_UNSUPPORTED;
   cudaStream_t s = (cudaStream_t)stream;
-  if (hd == 128) return launch2<128>(mk, mv, q, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
-  return launch2<64>(mk, mv, q, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
+  if (hd == 128) return so.dist ? launch2<128, true>(mk, mv, q, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s)
+                       : launch2<128, false>(mk, mv, q, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
+  return so.dist ? launch2<64, true>(mk, mv, q, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s)
+         : launch2<64, false>(mk, mv, q, block_table, table_stride, items, n_items, out, H, G, page_tokens, window, scale_log2, so, pages_cap, status, s);
 }
 
